@@ -4,3 +4,4 @@ from . import pedorax  # noqa: F401
 from . import putelix  # noqa: F401
 from . import roritar  # noqa: F401
 from . import mafuzen  # noqa: F401
+from . import pivinex  # noqa: F401

@@ -22,6 +22,8 @@ grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
                       const TW* __restrict__ w, int n_tokens, int a_stride, int a_off,
                       int a_gstride, int groups, int n, int k) {
   extern __shared__ float s_a[];                    // [GL_TT][k]
+  pdl_trigger();
+  pdl_wait();
   __shared__ float s_part[GL_THREADS / 32][GL_TT][GL_COLS];
   const int t0 = blockIdx.x * GL_TT;
   const int g = blockIdx.y;
@@ -77,6 +79,8 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
                           int a_off, int a_gstride, int groups, int N, int K, int vec) {
   __shared__ __align__(16) __nv_bfloat16 s_a[2][SPLIT][TM * TS];
   __shared__ __align__(16) __nv_bfloat16 s_b[2][TN * TS];
+  pdl_trigger();
+  pdl_wait();
   const int t0 = blockIdx.x * TM, n0 = blockIdx.y * TN, g = blockIdx.z;
   const int rows = min(TM, n_tokens - t0), ncols = min(TN, N - n0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -203,21 +207,21 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
   if (smem > 200 * 1024) return HS_ERR_UNSUPPORTED;
   dim3 grid((n_tokens + hs::GL_TT - 1) / hs::GL_TT, groups, (n + hs::GL_COLS - 1) / hs::GL_COLS);
   cudaStream_t st = (cudaStream_t)stream;
+  cudaError_t e = cudaSuccess;
 #define HS_GL(TW, TO)                                                                         \
   do {                                                                                        \
     auto kern = hs::grouped_linear_kernel<TW, TO>;                                            \
     if (smem > 48 * 1024)                                                                     \
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
-    kern<<<grid, hs::GL_THREADS, smem, st>>>((TO*)out, a, (const TW*)w, n_tokens, a_stride,  \
-                                             a_off, a_gstride, groups, n, k);                 \
+    e = hs_launch(kern, grid, dim3(hs::GL_THREADS), smem, st, hs_pdl_enabled(), (TO*)out, a, \
+                  (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k);          \
   } while (0)
   if (w_dtype == HS_DT_F32 && out_dtype == HS_DT_F32) HS_GL(float, float);
   else if (w_dtype == HS_DT_BF16 && out_dtype == HS_DT_F32) HS_GL(__nv_bfloat16, float);
   else if (w_dtype == HS_DT_BF16 && out_dtype == HS_DT_BF16) HS_GL(__nv_bfloat16, __nv_bfloat16);
   else return HS_ERR_UNSUPPORTED;
 #undef HS_GL
-  HS_LAUNCH_CHECK();
-  return HS_OK;
+  return e == cudaSuccess ? HS_OK : (int)e;
 }
 
 // The tensor-core form: weights [groups, n, k] bfloat16; k a multiple of 32.  Returns
@@ -232,22 +236,22 @@ HS_EXPORT int hs_grouped_linear_mma(void* out, const float* a, const void* w_nk,
   const int vec = a_stride % 4 == 0 && a_off % 4 == 0 && a_gstride % 4 == 0 && !((uintptr_t)a & 15);
   dim3 grid((n_tokens + hs::TM - 1) / hs::TM, (n + hs::TN - 1) / hs::TN, groups);
   cudaStream_t st = (cudaStream_t)stream;
+  const bool pdl = hs_pdl_enabled();
+  const __nv_bfloat16* w = (const __nv_bfloat16*)w_nk;
+  cudaError_t e = cudaSuccess;
   if (out_dtype == HS_DT_F32 && split == 3)
-    hs::grouped_linear_mma_kernel<float, 3><<<grid, 128, 0, st>>>(
-        (float*)out, a, (const __nv_bfloat16*)w_nk, n_tokens, a_stride, a_off, a_gstride, groups,
-        n, k, vec);
+    e = hs_launch(hs::grouped_linear_mma_kernel<float, 3>, grid, dim3(128), 0, st, pdl, (float*)out,
+                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec);
   else if (split == 3)
     return HS_ERR_UNSUPPORTED;
   else if (out_dtype == HS_DT_F32)
-    hs::grouped_linear_mma_kernel<float, 1><<<grid, 128, 0, st>>>(
-        (float*)out, a, (const __nv_bfloat16*)w_nk, n_tokens, a_stride, a_off, a_gstride, groups,
-        n, k, vec);
+    e = hs_launch(hs::grouped_linear_mma_kernel<float, 1>, grid, dim3(128), 0, st, pdl, (float*)out,
+                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec);
   else if (out_dtype == HS_DT_BF16)
-    hs::grouped_linear_mma_kernel<__nv_bfloat16, 1><<<grid, 128, 0, st>>>(
-        (__nv_bfloat16*)out, a, (const __nv_bfloat16*)w_nk, n_tokens, a_stride, a_off, a_gstride,
-        groups, n, k, vec);
+    e = hs_launch(hs::grouped_linear_mma_kernel<__nv_bfloat16, 1>, grid, dim3(128), 0, st, pdl,
+                  (__nv_bfloat16*)out, a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k,
+                  vec);
   else
     return HS_ERR_UNSUPPORTED;
-  HS_LAUNCH_CHECK();
-  return HS_OK;
+  return e == cudaSuccess ? HS_OK : (int)e;
 }

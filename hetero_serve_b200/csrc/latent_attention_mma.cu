@@ -1,8 +1,8 @@
 // Attention over a shared latent for prompt portions, on the tensor cores (mma.sync m16n8k16,
 // bfloat16 operands, float32 accumulators).  Same mathematics as latent_attention.cu:
 //
-//   score(i, j) = (qa_i . c_j + qr_i . kr_j) * scale  (j <= i),  softmax with a sink per head,
-//   out_lat     = sum_j weight_j c_j
+//   score(i, j) = (qa_i . c_j + qr_i . kr_j) * scale  (j <= i, with a window i - j < window),
+//   softmax (with a sink per head, if there are sinks),  out_lat = sum_j weight_j c_j
 //
 // Because every head of a token reads the same cache rows, a block's 64 query rows are (token,
 // head) pairs of consecutive tokens of ONE request: rows = token-major, head-minor, cut from a
@@ -42,7 +42,7 @@ latent_prefill_mma_kernel(float* __restrict__ out, const float* __restrict__ qa,
                           const int* __restrict__ plan, int tiles_off, int n_heads, int R, int P,
                           int qr_stride, int qr_hstride, int qr_off, float scale, int page_size,
                           int num_pages, int max_pages, int* status,
-                          const float* __restrict__ freq, int rot_dims) {
+                          const float* __restrict__ freq, int rot_dims, int window) {
   extern __shared__ __align__(16) __nv_bfloat16 sm_b[];
   if ((int)blockIdx.x >= plan[1]) return;
   const int* tile = plan + tiles_off + 4 * blockIdx.x;
@@ -95,8 +95,8 @@ latent_prefill_mma_kernel(float* __restrict__ out, const float* __restrict__ qa,
     const int tl = row_ok[x] ? row / n_heads : 0;
     row_head[x] = row_ok[x] ? row - tl * n_heads : 0;
     row_pos[x] = pos_first + tl;
-    m[x] = sink[row_head[x]];                     // the sink opens the running softmax
-    l[x] = tq == 0 ? 1.f : 0.f;                   // its weight 1 is counted once a row
+    m[x] = sink ? sink[row_head[x]] : -INFINITY;  // the sink opens the running softmax
+    l[x] = sink && tq == 0 ? 1.f : 0.f;           // its weight 1 is counted once a row
   }
   float acc_o[NTM][4];
 #pragma unroll
@@ -107,7 +107,9 @@ latent_prefill_mma_kernel(float* __restrict__ out, const float* __restrict__ qa,
   const int last_row = min(n_rows, row_lo + LM_ROWS) - 1;
   const int pos_max = pos_first + last_row / n_heads;        // the block's newest key
   const bool vec = (W & 7) == 0;
-  for (int base = 0; base <= pos_max; base += LM_KEYS) {
+  // the oldest key the block's first row sees: rows before it are not looked up
+  const int pos_min = window > 0 ? max(0, pos_first + row_lo / n_heads + 1 - window) : 0;
+  for (int base = pos_min / LM_KEYS * LM_KEYS; base <= pos_max; base += LM_KEYS) {
     __syncthreads();                              // sQ is set / the tile before has been used
     const int nk = min(LM_KEYS, pos_max + 1 - base);
     for (int j = warp; j < LM_KEYS; j += (blockDim.x >> 5)) {
@@ -115,7 +117,7 @@ latent_prefill_mma_kernel(float* __restrict__ out, const float* __restrict__ qa,
       const int kp = base + j;
       const int pi = kp / page_size;
       int page = -1;
-      if (j < nk) {
+      if (j < nk && kp >= pos_min) {
         page = pi < max_pages ? table[(size_t)req * max_pages + pi] : -1;
         if (page < 0 || page >= num_pages) {
           if (lane == 0) atomicOr(status, HS_STATUS_BAD_PAGE);
@@ -162,7 +164,7 @@ latent_prefill_mma_kernel(float* __restrict__ out, const float* __restrict__ qa,
       for (int c = 0; c < 4; ++c) {
         const int x = c >> 1;
         const int kp = base + 8 * j + 2 * tq + (c & 1);
-        const bool ok = row_ok[x] && kp <= row_pos[x];
+        const bool ok = row_ok[x] && kp <= row_pos[x] && (window <= 0 || row_pos[x] - kp < window);
         acc_s[j][c] = ok ? acc_s[j][c] * scale : -INFINITY;
         mx[x] = fmaxf(mx[x], acc_s[j][c]);
       }
@@ -172,15 +174,16 @@ latent_prefill_mma_kernel(float* __restrict__ out, const float* __restrict__ qa,
       mx[x] = fmaxf(mx[x], __shfl_xor_sync(0xffffffffu, mx[x], 1));
       mx[x] = fmaxf(mx[x], __shfl_xor_sync(0xffffffffu, mx[x], 2));
       const float m_new = fmaxf(m[x], mx[x]);
-      corr[x] = expf(m[x] - m_new);
+      corr[x] = m_new == -INFINITY ? 1.f : expf(m[x] - m_new);   // nothing visible so far
       m[x] = m_new;
       l[x] *= corr[x];
     }
     uint32_t pa[2][4];                            // P as the A operand of two steps of 16 keys
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const float p0 = expf(acc_s[j][0] - m[0]), p1 = expf(acc_s[j][1] - m[0]);
-      const float p2 = expf(acc_s[j][2] - m[1]), p3 = expf(acc_s[j][3] - m[1]);
+      const float m0 = m[0] == -INFINITY ? 0.f : m[0], m1 = m[1] == -INFINITY ? 0.f : m[1];
+      const float p0 = expf(acc_s[j][0] - m0), p1 = expf(acc_s[j][1] - m0);
+      const float p2 = expf(acc_s[j][2] - m1), p3 = expf(acc_s[j][3] - m1);
       l[0] += p0 + p1;
       l[1] += p2 + p3;
       pa[j >> 1][(j & 1) * 2] = pack_bf16(p0, p1);
@@ -233,8 +236,10 @@ HS_EXPORT int hs_latent_prefill_mma(float* out, const float* qa, const float* qr
                                     const int* plan, int tiles_off, int tile_cap, int n_heads,
                                     int R, int P, int qr_stride, int qr_hstride, int qr_off,
                                     float scale, int page_size, int num_pages, int max_pages,
-                                    int* status, const float* freq, int rot_dims, void* stream) {
-  if (!out || !qa || !qr || !pool || !table || !sink || !plan || !status) return HS_ERR_ARGUMENT;
+                                    int* status, const float* freq, int rot_dims, int window,
+                                    void* stream) {
+  if (!out || !qa || !qr || !pool || !table || !plan || !status || window < 0)
+    return HS_ERR_ARGUMENT;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > P || (rot_dims && !freq)) return HS_ERR_ARGUMENT;
   if (R <= 0 || R % 16 || R > 512 || P < 0 || n_heads <= 0 || page_size <= 0)
     return HS_ERR_UNSUPPORTED;
@@ -254,7 +259,7 @@ HS_EXPORT int hs_latent_prefill_mma(float* out, const float* qa, const float* qr
     kern<<<grid, 128 * halves, smem, st>>>(out, qa, qr, (const __nv_bfloat16*)pool, table,     \
                                            sink, plan, tiles_off, n_heads, R, P, qr_stride,    \
                                            qr_hstride, qr_off, scale, page_size, num_pages,    \
-                                           max_pages, status, freq, rot_dims);                 \
+                                           max_pages, status, freq, rot_dims, window);             \
   } while (0)
   if (per <= 128) HS_LM(16);
   else HS_LM(32);

@@ -12,6 +12,14 @@
 // (the lower index wins a tie) and weighted by the softmax over the chosen logits alone; and a
 // second expert activation (act 1): y = silu(W_g h) * (W_u h), no limit.
 //
+// A third rule (route_softmax): s = softmax(z) over all experts in float32; the `top` largest of
+// s + correction are chosen (the lower index wins a tie) and weigh s * scale (neither corrected
+// nor renormalised).
+//
+// Identity experts: choices E .. E + n_identity - 1 (behind the E experts that have matrices) add
+// weight * h itself, in the launch that adds the experts' weighted rows; a choice outside both
+// ranges adds nothing.  With `accumulate` 0 that launch writes the sum instead of adding it to x.
+//
 // Expert matrices are stacked as they are stored: gate / up [E, ff, width], down [E, width, ff]
 // (the summed index runs fastest).  Two paths:
 //   * few (token, expert) pairs, and all of float32: every pair streams its expert's rows, one
@@ -194,6 +202,77 @@ moe_route_top_kernel(int* __restrict__ sel_idx, float* __restrict__ sel_w,
   }
 }
 
+// z handed in: a warp chooses for a token (`blockDim.x / 32` tokens a block); else one block per
+// token forms the logits first and its warp 0 chooses.  The logits lie in shared memory, the
+// statistics of the softmax are formed in an order fixed by E.
+template <typename TH>
+__global__ void __launch_bounds__(256)
+moe_route_softmax_kernel(int* __restrict__ sel_idx, float* __restrict__ sel_w,
+                         const TH* __restrict__ h, const float* __restrict__ w_router,
+                         const float* __restrict__ correction, const int* __restrict__ tok_req,
+                         int n_tokens, int width, int E, int top, float scale,
+                         const float* __restrict__ z_in) {
+  extern __shared__ float smem[];
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* s_s;                       // [E] logits, then scores
+  int t;
+  if (z_in) {
+    t = blockIdx.x * (blockDim.x >> 5) + warp;
+    if (t >= n_tokens || tok_req[t] < 0) return;
+    s_s = smem + (size_t)warp * 2 * E;
+    for (int e = lane; e < E; e += 32) s_s[e] = z_in[(size_t)t * E + e];
+  } else {
+    t = blockIdx.x;
+    if (tok_req[t] < 0) return;
+    float* s_h = smem + 2 * E;      // [width]
+    s_s = smem;
+    for (int k = threadIdx.x; k < width; k += blockDim.x) s_h[k] = to_f(h[(size_t)t * width + k]);
+    __syncthreads();
+    for (int e = warp; e < E; e += blockDim.x / 32) {
+      const float z = row_dot(w_router + (size_t)e * width, s_h, width, lane);
+      if (lane == 0) s_s[e] = z;
+    }
+    __syncthreads();
+    if (warp != 0) return;
+  }
+  __syncwarp();
+  float* s_c = s_s + E;             // [E] what the choice looks at (-inf once taken)
+  float m = -INFINITY;
+  for (int e = lane; e < E; e += 32) m = fmaxf(m, s_s[e]);
+  m = warp_max(m);
+  float total = 0.f;
+  for (int e = lane; e < E; e += 32) {
+    const float v = expf(s_s[e] - m);
+    s_s[e] = v;
+    total += v;
+  }
+  total = warp_sum(total);
+  for (int e = lane; e < E; e += 32) {
+    const float v = s_s[e] / total;
+    s_s[e] = v;
+    s_c[e] = v + (correction ? correction[e] : 0.f);
+  }
+  __syncwarp();
+  for (int round = 0; round < top; ++round) {
+    float bv = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const float v = s_c[e];
+      if (v > bv) { bv = v; bi = e; }
+    }
+    warp_argmax(bv, bi);
+    if (lane == 0) {
+      const bool ok = bi < E;
+      sel_idx[(size_t)t * top + round] = ok ? bi : -1;
+      sel_w[(size_t)t * top + round] = ok ? s_s[bi] * scale : 0.f;
+      if (ok) s_c[bi] = -INFINITY;                       // taken
+    }
+    __syncwarp();
+  }
+}
+
 // act 0: the clamped form above; act 1: silu(g) * u; act 2: relu(u)^2 (an expert without a gate
 // matrix)
 __device__ __forceinline__ float expert_act(float g, float u, float limit, int act) {
@@ -263,6 +342,8 @@ moe_gate_up_rows_kernel(float* __restrict__ y, const TW* __restrict__ h,
                         const int* __restrict__ sel_idx, const int* __restrict__ tok_req,
                         int width, int ff, int top, int E, float limit, int act) {
   extern __shared__ __align__(16) float s_h[];         // [width]
+  pdl_trigger();
+  pdl_wait();
   const int pair = blockIdx.x;
   const int t = pair / top;
   if (tok_req[t] < 0) return;
@@ -297,14 +378,18 @@ __global__ void __launch_bounds__(GEMV_THREADS)
 moe_down_rows_kernel(float* __restrict__ x, const float* __restrict__ y,
                      const TW* __restrict__ w_down, const int* __restrict__ sel_idx,
                      const float* __restrict__ sel_w, const int* __restrict__ tok_req, int width,
-                     int ff, int top, int E) {
+                     int ff, int top, int E, const TW* __restrict__ h, int n_identity,
+                     int accumulate) {
   extern __shared__ __align__(16) float s_y[];         // [top][ff4]: rows padded to 16 bytes
+  pdl_trigger();
+  pdl_wait();
   const int t = blockIdx.x;
   if (tok_req[t] < 0) return;
   const int ff4 = (ff + 3) & ~3;
   for (int i = threadIdx.x; i < top * ff4; i += GEMV_THREADS) {
     const int k = i / ff4, f = i - k * ff4;
-    s_y[i] = f < ff ? y[((size_t)t * top + k) * ff + f] : 0.f;
+    const int e = sel_idx[(size_t)t * top + k];           // other choices left nothing in y
+    s_y[i] = f < ff && e >= 0 && e < E ? y[((size_t)t * top + k) * ff + f] : 0.f;
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -356,9 +441,15 @@ moe_down_rows_kernel(float* __restrict__ x, const float* __restrict__ y,
       }
 #pragma unroll
       for (int i = 0; i < MAX_TOP_AT_ONCE; ++i)
-        if (k0 + i < top) sum = fmaf(sel_w[(size_t)t * top + k0 + i], acc[i], sum);
+        if (k0 + i < top) {
+          if (n_identity) {
+            const int e = sel_idx[(size_t)t * top + k0 + i];
+            if (e >= E && e < E + n_identity) acc[i] = to_f(h[(size_t)t * width + n]);
+          }
+          sum = fmaf(sel_w[(size_t)t * top + k0 + i], acc[i], sum);
+        }
     }
-    if (lane == 0) x[(size_t)t * width + n] += sum;
+    if (lane == 0) x[(size_t)t * width + n] = accumulate ? x[(size_t)t * width + n] + sum : sum;
   }
 }
 
@@ -373,6 +464,8 @@ moe_sort_kernel(int* __restrict__ work, int* __restrict__ pair_pos, int* __restr
                 const int* __restrict__ sel_idx, const int* __restrict__ tok_req, int n_tokens,
                 int top, int E, int max_tiles) {
   extern __shared__ int s_cnt[];             // [E] counts, then [E] cursors
+  pdl_trigger();
+  pdl_wait();
   int* s_cur = s_cnt + E;
   for (int e = threadIdx.x; e < E; e += SORT_THREADS) s_cnt[e] = 0;
   __syncthreads();
@@ -427,6 +520,8 @@ moe_tiles_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ a,
                  int max_tiles, int N, int K, float limit, int act) {
   __shared__ __align__(16) __nv_bfloat16 s_a[2][TM * TS];
   __shared__ __align__(16) __nv_bfloat16 s_b[NB][2][TN * TS];
+  pdl_trigger();
+  pdl_wait();
   const int tile = blockIdx.x;
   if (tile >= work[0]) return;
   const int e = work[1 + 2 * E + tile];
@@ -517,20 +612,31 @@ moe_tiles_kernel(void* __restrict__ out, const __nv_bfloat16* __restrict__ a,
       }
 }
 
-// x[t] += sum_k weight_k * rows[pair_pos[t, k]], experts in the order they were chosen
+// x[t] (+)= sum_k weight_k * rows[pair_pos[t, k]], experts in the order they were chosen
 __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restrict__ rows,
                                    const int* __restrict__ pair_pos,
                                    const float* __restrict__ sel_w,
-                                   const int* __restrict__ tok_req, int width, int top) {
+                                   const int* __restrict__ tok_req, int width, int top,
+                                   const int* __restrict__ sel_idx,
+                                   const __nv_bfloat16* __restrict__ h, int E, int n_identity,
+                                   int accumulate) {
+  pdl_trigger();
+  pdl_wait();
   const int t = blockIdx.x;
   if (tok_req[t] < 0) return;
   for (int n = threadIdx.x; n < width; n += blockDim.x) {
     float sum = 0.f;
     for (int k = 0; k < top; ++k) {
       const int pos = pair_pos[(size_t)t * top + k];
-      if (pos >= 0) sum = fmaf(sel_w[(size_t)t * top + k], rows[(size_t)pos * width + n], sum);
+      if (pos >= 0) {
+        sum = fmaf(sel_w[(size_t)t * top + k], rows[(size_t)pos * width + n], sum);
+      } else if (n_identity) {
+        const int e = sel_idx[(size_t)t * top + k];
+        if (e >= E && e < E + n_identity)
+          sum = fmaf(sel_w[(size_t)t * top + k], to_f(h[(size_t)t * width + n]), sum);
+      }
     }
-    x[(size_t)t * width + n] += sum;
+    x[(size_t)t * width + n] = accumulate ? x[(size_t)t * width + n] + sum : sum;
   }
 }
 
@@ -579,6 +685,33 @@ HS_EXPORT int hs_moe_route_top(int* sel_idx, float* sel_w, const void* h, const 
   else if (h_dtype == HS_DT_BF16)
     e = hs_launch(hs::moe_route_top_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), smem, st, hs_pdl_enabled(), sel_idx, sel_w,
                   (const __nv_bfloat16*)h, w_router, bias, tok_req, width, E, top, z_in);
+  else
+    return HS_ERR_UNSUPPORTED;
+  return e == cudaSuccess ? HS_OK : (int)e;
+}
+
+HS_EXPORT int hs_moe_route_softmax(int* sel_idx, float* sel_w, const void* h,
+                                   const float* w_router, const float* correction,
+                                   const int* tok_req, int n_tokens, int width, int E, int top,
+                                   float scale, int h_dtype, const float* z_in, void* stream) {
+  if (!sel_idx || !sel_w || !h || !w_router || !tok_req) return HS_ERR_ARGUMENT;
+  if (width <= 0 || E <= 0 || top <= 0 || top > E) return HS_ERR_UNSUPPORTED;
+  if (n_tokens <= 0) return HS_OK;
+  int warps = (E + 3) / 4;                       // four experts a warp, up to eight warps
+  warps = z_in ? 4 : (warps < 1 ? 1 : (warps > 8 ? 8 : warps));
+  const size_t smem = (z_in ? (size_t)warps * 2 * E : (size_t)2 * E + width) * sizeof(float);
+  if (smem > 48 * 1024) return HS_ERR_UNSUPPORTED;
+  const dim3 grid(z_in ? (n_tokens + warps - 1) / warps : n_tokens);
+  cudaStream_t st = (cudaStream_t)stream;
+  cudaError_t e = cudaSuccess;
+  if (h_dtype == HS_DT_F32)
+    e = hs_launch(hs::moe_route_softmax_kernel<float>, grid, dim3(32 * warps), smem, st,
+                  hs_pdl_enabled(), sel_idx, sel_w, (const float*)h, w_router, correction, tok_req,
+                  n_tokens, width, E, top, scale, z_in);
+  else if (h_dtype == HS_DT_BF16)
+    e = hs_launch(hs::moe_route_softmax_kernel<__nv_bfloat16>, grid, dim3(32 * warps), smem, st,
+                  hs_pdl_enabled(), sel_idx, sel_w, (const __nv_bfloat16*)h, w_router, correction,
+                  tok_req, n_tokens, width, E, top, scale, z_in);
   else
     return HS_ERR_UNSUPPORTED;
   return e == cudaSuccess ? HS_OK : (int)e;
@@ -646,12 +779,15 @@ HS_EXPORT int hs_moe_experts(float* x, float* y, const void* h, const void* w_ga
                              const void* w_up, const void* w_down, const int* sel_idx,
                              const float* sel_w, const int* tok_req, int n_tokens, int width,
                              int ff, int top, int E, float limit, int act_kind, int dtype, int* ints,
-                             void* rows, void* stream) {
+                             void* rows, int n_identity, int accumulate, void* stream) {
   if (!x || !h || !w_up || !w_down || !sel_idx || !sel_w || !tok_req || (!w_gate && act_kind != 2))
     return HS_ERR_ARGUMENT;
-  if (width <= 0 || ff <= 0 || top <= 0 || E <= 0 || act_kind < 0 || act_kind > 2) return HS_ERR_UNSUPPORTED;
+  if (width <= 0 || ff <= 0 || top <= 0 || E <= 0 || act_kind < 0 || act_kind > 2 || n_identity < 0)
+    return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
   cudaStream_t st = (cudaStream_t)stream;
+  const bool pdl = hs_pdl_enabled();
+  cudaError_t e;
   if (ints && rows) {
     long long need_i = 0, need_b = 0;
     hs_moe_sorted_scratch(n_tokens, width, ff, top, E, dtype, &need_i, &need_b);
@@ -663,27 +799,30 @@ HS_EXPORT int hs_moe_experts(float* x, float* y, const void* h, const void* w_ga
     int* row_token = pair_pos + pairs;
     __nv_bfloat16* act = (__nv_bfloat16*)rows;
     float* down = (float*)((char*)rows + (((size_t)pairs * ff * 2 + 255) / 256) * 256);
-    hs::moe_sort_kernel<<<1, hs::SORT_THREADS, 2 * E * sizeof(int), st>>>(
-        work, pair_pos, row_token, sel_idx, tok_req, n_tokens, top, E, max_tiles);
-    HS_LAUNCH_CHECK();
+    e = hs_launch(hs::moe_sort_kernel, dim3(1), dim3(hs::SORT_THREADS), 2 * E * sizeof(int), st,
+                  pdl, work, pair_pos, row_token, sel_idx, tok_req, n_tokens, top, E, max_tiles);
+    if (e != cudaSuccess) return (int)e;
     const __nv_bfloat16* hb = (const __nv_bfloat16*)h;
+    const __nv_bfloat16* none = nullptr;
+    const dim3 g1(max_tiles, (ff + hs::TN - 1) / hs::TN);
     if (w_gate)
-      hs::moe_tiles_kernel<2, true><<<dim3(max_tiles, (ff + hs::TN - 1) / hs::TN), 128, 0, st>>>(
-          act, hb, (const __nv_bfloat16*)w_gate, (const __nv_bfloat16*)w_up, work, row_token, E,
-          max_tiles, ff, width, limit, act_kind);
+      e = hs_launch(hs::moe_tiles_kernel<2, true>, g1, dim3(128), 0, st, pdl, (void*)act, hb,
+                    (const __nv_bfloat16*)w_gate, (const __nv_bfloat16*)w_up, (const int*)work,
+                    (const int*)row_token, E, max_tiles, ff, width, limit, act_kind);
     else
-      hs::moe_tiles_kernel<1, true, true><<<dim3(max_tiles, (ff + hs::TN - 1) / hs::TN), 128, 0, st>>>(
-          act, hb, (const __nv_bfloat16*)w_up, nullptr, work, row_token, E, max_tiles, ff, width,
-          limit, act_kind);
-    HS_LAUNCH_CHECK();
-    hs::moe_tiles_kernel<1, false><<<dim3(max_tiles, (width + hs::TN - 1) / hs::TN), 128, 0, st>>>(
-        down, act, (const __nv_bfloat16*)w_down, nullptr, work, row_token, E, max_tiles, width,
-        ff, limit, act_kind);
-    HS_LAUNCH_CHECK();
-    hs::moe_combine_kernel<<<n_tokens, 256, 0, st>>>(x, down, pair_pos, sel_w, tok_req, width,
-                                                     top);
-    HS_LAUNCH_CHECK();
-    return HS_OK;
+      e = hs_launch(hs::moe_tiles_kernel<1, true, true>, g1, dim3(128), 0, st, pdl, (void*)act, hb,
+                    (const __nv_bfloat16*)w_up, none, (const int*)work, (const int*)row_token, E,
+                    max_tiles, ff, width, limit, act_kind);
+    if (e != cudaSuccess) return (int)e;
+    e = hs_launch(hs::moe_tiles_kernel<1, false>, dim3(max_tiles, (width + hs::TN - 1) / hs::TN),
+                  dim3(128), 0, st, pdl, (void*)down, (const __nv_bfloat16*)act,
+                  (const __nv_bfloat16*)w_down, none, (const int*)work, (const int*)row_token, E,
+                  max_tiles, width, ff, limit, act_kind);
+    if (e != cudaSuccess) return (int)e;
+    e = hs_launch(hs::moe_combine_kernel, dim3(n_tokens), dim3(256), 0, st, pdl, x,
+                  (const float*)down, (const int*)pair_pos, sel_w, tok_req, width, top, sel_idx, hb,
+                  E, n_identity, accumulate);
+    return e == cudaSuccess ? HS_OK : (int)e;
   }
   if (!y) return HS_ERR_ARGUMENT;
   const size_t smem_h = (size_t)width * sizeof(float);
@@ -699,17 +838,17 @@ HS_EXPORT int hs_moe_experts(float* x, float* y, const void* h, const void* w_ga
       cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_h);      \
     if (smem_y > 48 * 1024)                                                                    \
       cudaFuncSetAttribute(k2, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_y);      \
-    k1<<<g1, hs::GEMV_THREADS, smem_h, st>>>(y, (const TW*)h, (const TW*)w_gate,               \
-                                             (const TW*)w_up, sel_idx, tok_req, width, ff,     \
-                                             top, E, limit, act_kind);                         \
-    HS_LAUNCH_CHECK();                                                                         \
-    k2<<<g2, hs::GEMV_THREADS, smem_y, st>>>(x, y, (const TW*)w_down, sel_idx, sel_w, tok_req, \
-                                             width, ff, top, E);                               \
+    e = hs_launch(k1, g1, dim3(hs::GEMV_THREADS), smem_h, st, pdl, y, (const TW*)h,            \
+                  (const TW*)w_gate, (const TW*)w_up, sel_idx, tok_req, width, ff, top, E,     \
+                  limit, act_kind);                                                            \
+    if (e != cudaSuccess) return (int)e;                                                       \
+    e = hs_launch(k2, g2, dim3(hs::GEMV_THREADS), smem_y, st, pdl, x, (const float*)y,         \
+                  (const TW*)w_down, sel_idx, sel_w, tok_req, width, ff, top, E, (const TW*)h, \
+                  n_identity, accumulate);                                                     \
   } while (0)
   if (dtype == HS_DT_F32) HS_MOE(float);
   else if (dtype == HS_DT_BF16) HS_MOE(__nv_bfloat16);
   else return HS_ERR_UNSUPPORTED;
 #undef HS_MOE
-  HS_LAUNCH_CHECK();
-  return HS_OK;
+  return e == cudaSuccess ? HS_OK : (int)e;
 }

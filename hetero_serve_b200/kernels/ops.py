@@ -202,16 +202,18 @@ def _declare(lib) -> None:
         "hs_rotary_pairs": [P, P, P, P, I, I, I, I, I, I, P],
         "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P],
         "hs_grouped_linear_mma": [P, P, P, I, I, I, I, I, I, I, I, I, P],
-        "hs_latent_append": [P, P, P, P, P, P, I, I, I, I, I, F, I, I, I, I, P, P, I, P],
+        "hs_latent_append": [P, P, P, P, P, P, I, I, I, I, I, F, I, I, I, I, P, P, I, P, P, I, I,
+                             P],
         "hs_latent_attention": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, P, I,
-                                P, P, I, P, P],
+                                P, P, I, P, I, P],
         "hs_latent_prefill_mma": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, P,
-                                  I, P],
+                                  I, I, P],
         "hs_delta_prepare": [P] * 15 + [I] * 9 + [P, P],
         "hs_delta_recurrence": [P] * 10 + [I] * 8 + [P],
         "hs_delta_finish": [P, P, P, P, P, P, I, F, I, I, I, I, I, I, I, I, P, P],
         "hs_moe_route": [P, P, P, P, P, I, I, I, I, I, I, I, P, P],
-        "hs_moe_experts": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, F, I, I, P, P, P],
+        "hs_moe_experts": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, F, I, I, P, P, I, I, P],
+        "hs_moe_route_softmax": [P, P, P, P, P, P, I, I, I, I, F, I, P, P],
         "hs_moe_route_top": [P, P, P, P, P, P, I, I, I, I, I, P, P],
         "hs_rms_norm": [P, P, P, P, I, I, F, I, P, I, I, I, P],
         "hs_rms_norm_add": [P, P, P, P, P, P, F, P, I, I, F, F, I, P, P, F, P],
@@ -235,6 +237,8 @@ def _declare(lib) -> None:
                               I, P, P, P, P],
         "hs_span_attention_prefill": [P, P, P, P, I, I, P, P, I, P, P, P, I, I, F, I, I, I, I, I, I,
                                       F, I, P, P],
+        "hs_embed_norm": [P, P, P, P, P, I, I, I, I, P, I, P, P, F, P, P, P, F, I, P, P],
+        "hs_residual_mix": [P, P, P, P, P, P, I, I, P, P, P, F, I, P],
         "hs_layernorm_add": [P, P, P, P, F, P, P, P, F, I, I, I, P],
         "hs_learned_act_xielu": [P, P, ctypes.c_longlong, F, F, I, P],
         "hs_scale_softcap": [P, ctypes.c_longlong, F, F, P],
@@ -1095,12 +1099,15 @@ class CudaOps:
 
     # -- attention over a shared latent ---------------------------------------------------
     def latent_append(self, pool, proj, norm_w, table, tok_pos, tok_req, *, c_offset, rank,
-                      rot_dim, eps, page_size, status, freq=None, rot_dims=0):
+                      rot_dim, eps, page_size, status, freq=None, rot_dims=0, q_out=None,
+                      q_norm=None, q_offset=0):
         """Cache row of each token: ``[rms_norm(proj[t, c_offset : +rank]) * norm_w |
         proj[t, c_offset + rank : + rot_dim]]``; with ``freq`` the first ``rot_dims`` entries
         of the second part are rotated on the way (interleaved pairs, as ``rotary_pairs``),
         without it the part is taken as it stands.  ``pool`` is [pages, 1, 1, page_size,
-        rank + rot_dim]."""
+        rank + rot_dim].  With ``q_out`` [T, q_rank] (of the pool's type) the same launch also
+        leaves ``rms_norm(proj[t, q_offset : + q_rank]) * q_norm`` there: a latent the queries
+        come through."""
         _want(proj, "proj", torch.float32, 2)
         _want(pool, "pool", _FLOATS)
         _want(norm_w, "norm_w", torch.float32, 1)
@@ -1111,6 +1118,13 @@ class CudaOps:
             raise KernelError("latent_append: pool or norm weight does not fit rank + rot_dim")
         if c_offset + W > proj.shape[1] or tok_pos.shape[0] < n or tok_req.shape[0] < n:
             raise KernelError("latent_append: rows do not fit")
+        q_rank = 0
+        if q_out is not None:
+            _want(q_out, "q_out", pool.dtype, 2)
+            _want(q_norm, "q_norm", torch.float32, 1)
+            q_rank = q_out.shape[1]
+            if q_norm.shape[0] != q_rank or q_out.shape[0] < n or q_offset + q_rank > proj.shape[1]:
+                raise KernelError("latent_append: the query latent does not fit")
         self.launches += 1
         _check(self.lib.hs_latent_append(_ptr(pool), _ptr(proj), _ptr(norm_w), _ptr(table),
                                          _ptr(tok_pos), _ptr(tok_req), n, proj.shape[1],
@@ -1118,15 +1132,17 @@ class CudaOps:
                                          pool.numel() // (page_size * W), table.shape[1],
                                          _DT[pool.dtype], _ptr(status), _ptr(freq),
                                          int(rot_dims) if freq is not None else 0,
+                                         _ptr(q_out), _ptr(q_norm), int(q_offset), q_rank,
                                          self._stream()),
                "latent_append")
 
     def latent_attention(self, out, qa, qr, pool, table, tok_pos, tok_req, sink, *, n_heads,
                          rank, rot_dim, qr_head_stride, qr_offset, scale, page_size, status,
-                         freq=None, rot_dims=0, plan=None):
-        """Causal softmax attention with a sink over cache rows ``[c (rank) | kr (rot_dim)]``
-        shared by all heads: score = (qa[t,h] . c + qr[t,h] . kr) * scale, the denominator
-        also holds exp(sink[h]); ``out[t, h] = sum_j weight_j c_j`` ([T, n_heads * rank],
+                         freq=None, rot_dims=0, plan=None, window=0):
+        """Causal softmax attention over cache rows ``[c (rank) | kr (rot_dim)]`` shared by all
+        heads: score = (qa[t,h] . c + qr[t,h] . kr) * scale over every earlier position, or with
+        ``window`` the last ``window`` ones (the token itself among them); with ``sink`` the
+        denominator also holds exp(sink[h]) (None: it does not); ``out[t, h] = sum_j weight_j c_j`` ([T, n_heads * rank],
         float32).  ``qa`` [T, n_heads * rank] float32; head h's rotated query part is
         ``qr[t, qr_offset + h * qr_head_stride : + rot_dim]``; with ``freq`` it arrives
         unrotated and its first ``rot_dims`` entries are rotated as they are read.  With the
@@ -1138,14 +1154,17 @@ class CudaOps:
         _want(qr, "qr", torch.float32, 2)
         _want(pool, "pool", _FLOATS)
         _want(table, "table", torch.int32, 2)
-        _want(sink, "sink", torch.float32, 1)
+        if sink is not None:
+            _want(sink, "sink", torch.float32, 1)
         n = out.shape[0]
         W = rank + rot_dim
+        if window < 0:
+            raise KernelError("latent_attention: a window is not negative")
         if out.shape[1] != n_heads * rank or qa.shape[1] != n_heads * rank or qa.shape[0] < n:
             raise KernelError("latent_attention: out / qa are [T, n_heads * rank]")
         if qr.shape[0] < n or qr_offset + (n_heads - 1) * qr_head_stride + rot_dim > qr.shape[1]:
             raise KernelError("latent_attention: the rotated query parts exceed qr's row")
-        if pool.numel() % (page_size * W) or sink.shape[0] != n_heads:
+        if pool.numel() % (page_size * W) or (sink is not None and sink.shape[0] != n_heads):
             raise KernelError("latent_attention: pool or sink does not fit")
         rot = int(rot_dims) if freq is not None else 0
         n_pages = pool.numel() // (page_size * W)
@@ -1156,7 +1175,7 @@ class CudaOps:
                 _ptr(out), _ptr(qa), _ptr(qr), _ptr(pool), _ptr(table), _ptr(sink),
                 _ptr(plan.data), 4 + plan_decode_ints(plan.n_rows), plan.tile_cap, n_heads, rank,
                 rot_dim, qr.shape[1], int(qr_head_stride), int(qr_offset), float(scale),
-                page_size, n_pages, table.shape[1], _ptr(status), _ptr(freq), rot,
+                page_size, n_pages, table.shape[1], _ptr(status), _ptr(freq), rot, int(window),
                 self._stream())
             if code != -1:
                 _check(code, f"latent_prefill_mma(rank={rank},rot_dim={rot_dim})")
@@ -1168,6 +1187,8 @@ class CudaOps:
         # few tokens: the keys of each are split over several blocks so that the device fills
         blocks = n * -(-n_heads // 8)
         nsplit = 1 if blocks >= self.sm_count else min(16, -(-2 * self.sm_count // blocks))
+        if window > 0:                 # no more shares than tiles of 32 keys a window touches
+            nsplit = min(nsplit, (window + 30) // 32 + 1)
         if self.latent_splits is not None:
             nsplit = int(self.latent_splits)
         partial = None
@@ -1182,7 +1203,7 @@ class CudaOps:
             _ptr(sink), n, n_heads, rank, rot_dim, qr.shape[1], int(qr_head_stride),
             int(qr_offset), float(scale), page_size, n_pages,
             table.shape[1], _DT[pool.dtype], _ptr(status), nsplit, _ptr(partial), _ptr(freq),
-            rot, _ptr(listed), self._stream()),
+            rot, _ptr(listed), int(window), self._stream()),
             f"latent_attention(rank={rank},rot_dim={rot_dim})")
 
     # -- the gated delta rule ---------------------------------------------------------------
@@ -1266,7 +1287,7 @@ class CudaOps:
                f"moe_route(experts={E},top={top},groups={n_groups},keep={keep})")
 
     def moe_experts(self, x, y, h, w_gate, w_up, w_down, sel_idx, sel_w, tok_req, *, limit,
-                    act="clamped"):
+                    act="clamped", identity=0, fresh=False):
         """x += sum over a token's chosen experts of weight * W_down act(W_gate h, W_up h) with
         act(g, u) = min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, +-limit) + 1)
         (``act="clamped"``) or silu(g) * u (``act="silu"``, no limit), or W_down relu(W_up h)^2
@@ -1274,7 +1295,8 @@ class CudaOps:
         Expert matrices stacked as stored: gate / up [E, ff, width], down [E, width, ff]; ``y``
         is float32 scratch [T * top, ff].  Many pairs in bfloat16 are sorted by expert on the
         device and run as tiles on the tensor cores; few pairs, and float32, as one
-        matrix-vector product per pair."""
+        matrix-vector product per pair.  Choices E .. E + ``identity`` - 1 (behind the experts
+        with matrices) add weight * h.  With ``fresh`` the sum is written to x, not added."""
         _want(x, "x", torch.float32, 2)
         _want(y, "y", torch.float32, 2)
         _want(h, "h", _FLOATS, 2)
@@ -1306,7 +1328,8 @@ class CudaOps:
                                        _ptr(w_down), _ptr(sel_idx), _ptr(sel_w), _ptr(tok_req),
                                        T, width, ff, top, E, float(limit),
                                        EXPERT_ACTIVATIONS[act], _DT[h.dtype],
-                                       _ptr(ints), _ptr(rows), self._stream()),
+                                       _ptr(ints), _ptr(rows), int(identity), int(not fresh),
+                                       self._stream()),
                f"moe_experts(ff={ff})")
 
     def moe_route_top(self, sel_idx, sel_w, h, w_router, bias, tok_req, *, top, z=None):
@@ -1329,6 +1352,106 @@ class CudaOps:
                                          _ptr(bias), _ptr(tok_req), sel_idx.shape[0], width, E,
                                          top, _DT[h.dtype], _ptr(z), self._stream()),
                f"moe_route_top(experts={E},top={top})")
+
+    def moe_route_softmax(self, sel_idx, sel_w, h, w_router, correction, tok_req, *, top, scale,
+                          z=None):
+        """Per token: scores s = softmax(W_r h) over all outputs in float32, the ``top`` largest
+        of ``s + correction`` are chosen (the lower index wins a tie) with the weights
+        ``s * scale``.  ``z`` [T, outputs] float32, if given, holds ``W_r h``."""
+        _want(sel_idx, "sel_idx", torch.int32, 2)
+        _want(sel_w, "sel_w", torch.float32, 2)
+        _want(h, "h", _FLOATS, 2)
+        _want(w_router, "w_router", torch.float32, 2)
+        E, width = w_router.shape
+        if correction is not None:
+            _want(correction, "correction", torch.float32, 1)
+            if correction.shape[0] != E:
+                raise KernelError("moe_route_softmax: one correction per output of the router")
+        if h.shape[1] != width or sel_idx.shape[1] != top or sel_w.shape[1] != top:
+            raise KernelError("moe_route_softmax: shapes do not fit")
+        self.launches += 1
+        _check(self.lib.hs_moe_route_softmax(_ptr(sel_idx), _ptr(sel_w), _ptr(h), _ptr(w_router),
+                                             _ptr(correction), _ptr(tok_req), sel_idx.shape[0],
+                                             width, E, top, float(scale), _DT[h.dtype], _ptr(z),
+                                             self._stream()),
+               f"moe_route_softmax(outputs={E},top={top})")
+
+    # -- the stream around a parallel block -----------------------------------------------
+    def _norm_out(self, x, out, norm):
+        """The arguments of an optional layer norm of the new rows: ``norm = (weight, bias, eps)``."""
+        if (out is None) != (norm is None):
+            raise KernelError("out and norm come together")
+        if out is None:
+            return None, None, 0.0, 0
+        g, b, eps = norm
+        _want(out, "out", _FLOATS, 2)
+        for t, nm in ((g, "norm weight"), (b, "norm bias")):
+            if t is not None:
+                _want(t, nm, torch.float32, 1)
+                if t.shape[0] != x.shape[1]:
+                    raise KernelError(f"{nm}: length != width")
+        if tuple(out.shape) != tuple(x.shape):
+            raise KernelError("out and x have the same shape")
+        return g, b, float(eps), _DT[out.dtype]
+
+    def embed_norm(self, x, ids, req, table, weight, bias, eps, status, feedback=None, keep=None,
+                   out=None, norm=None):
+        """x[t] = layer_norm(table[ids[t]]) * weight (+ bias), rows with req[t] < 0 become zero;
+        ``keep`` (like x) receives a copy; with ``norm = (weight, bias, eps)`` ``out`` receives
+        the layer norm of the new rows (of the block that runs first).  ``feedback`` as in
+        `embed`."""
+        _want(x, "x", torch.float32, 2)
+        _want(table, "table", _FLOATS, 2)
+        n, width = x.shape
+        for t, nm in ((ids, "ids"), (req, "req")):
+            _want(t, nm, torch.int32, 1)
+            if t.shape[0] < n:
+                raise KernelError(f"{nm}: {t.shape[0]} entries for {n} rows")
+        _want(weight, "weight", torch.float32, 1)
+        if bias is not None:
+            _want(bias, "bias", torch.float32, 1)
+        if table.shape[1] != width or weight.shape[0] != width or \
+                (bias is not None and bias.shape[0] != width):
+            raise KernelError("embed_norm: widths of x, table, weight and bias differ")
+        if keep is not None:
+            _want(keep, "keep", torch.float32, 2)
+            if tuple(keep.shape) != (n, width):
+                raise KernelError("embed_norm: keep is shaped like x")
+        if feedback is not None:
+            _want(feedback, "feedback", torch.int32, 1)
+        g2, b2, eps2, out_dt = self._norm_out(x, out, norm)
+        self.launches += 1
+        _check(self.lib.hs_embed_norm(
+            _ptr(x), _ptr(keep), _ptr(ids), _ptr(req), _ptr(table), n, width, table.shape[0],
+            _DT[table.dtype], _ptr(feedback), 0 if feedback is None else feedback.shape[0],
+            _ptr(weight), _ptr(bias), float(eps), _ptr(out), _ptr(g2), _ptr(b2), eps2, out_dt,
+            _ptr(status), self._stream()), f"embed_norm(width={width})")
+
+    def residual_mix(self, x, y1=None, s1=None, y2=None, s2=None, again=None, out=None, norm=None):
+        """x += s1 * y1 + s2 * y2 (+ again): sublayer outputs (float32 blocks like x) times one
+        factor per column, and optionally a third block as it is; with ``norm = (weight, bias,
+        eps)`` ``out`` receives the layer norm of the new rows in its own type."""
+        _want(x, "x", torch.float32, 2)
+        n, width = x.shape
+        if y1 is None and y2 is None and again is None:
+            raise KernelError("residual_mix: nothing to add")
+        for y, s, nm in ((y1, s1, "1"), (y2, s2, "2")):
+            if (y is None) != (s is None):
+                raise KernelError("residual_mix: a block and its factors come together")
+            if y is not None:
+                _want(y, "y" + nm, torch.float32, 2)
+                _want(s, "s" + nm, torch.float32, 1)
+                if tuple(y.shape) != (n, width) or s.shape[0] != width:
+                    raise KernelError("residual_mix: shapes do not fit")
+        if again is not None:
+            _want(again, "again", torch.float32, 2)
+            if tuple(again.shape) != (n, width):
+                raise KernelError("residual_mix: shapes do not fit")
+        g, b, eps, out_dt = self._norm_out(x, out, norm)
+        self.launches += 1
+        _check(self.lib.hs_residual_mix(_ptr(x), _ptr(y1), _ptr(s1), _ptr(y2), _ptr(s2),
+                                        _ptr(again), n, width, _ptr(out), _ptr(g), _ptr(b), eps,
+                                        out_dt, self._stream()), f"residual_mix(width={width})")
 
     def gated_act(self, out, gu, h=None, w_s=None, tok_req=None, act="silu"):
         """out[t, f] = act(gu[t, f]) * gu[t, ff + f] (* sigmoid(h[t] . w_s), one number per

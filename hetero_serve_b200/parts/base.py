@@ -3,7 +3,7 @@
 A part is built from the parameters of its :class:`PartSpec` alone.  It says which
 checkpoint tensors it needs (:meth:`Part.tensor_requests`), receives them converted
 and on the device (:meth:`Part.bind`) and runs on a :class:`StepContext`
-(``hetero_serve_b200.engine.context``).  Five kinds exist:
+(``hetero_serve_b200.engine.context``).  Six kinds exist:
 
 ========  ==================================================================
 mixer     ``forward(ctx, h, x, cache)``: mixes information between the tokens
@@ -11,6 +11,8 @@ mixer     ``forward(ctx, h, x, cache)``: mixes information between the tokens
           residual stream ``x``.  Declares what it needs cached.
 feed      ``forward(ctx, h, x)``: per-token transform, added into ``x``.
 norm      ``forward(ctx, out, x, rows=None)``: normalises rows of ``x``.
+scale     ``factor``: a float32 vector [width] an arrangement multiplies a
+          sublayer's output with, column by column, before it is added.
 position  how positions enter: a table added at the embedding and/or a
           transform of queries and keys inside a mixer.
 embedding / head: token table at the input, logits at the output.
@@ -124,6 +126,10 @@ class Norm(Part):
         ctx.ops.linear(out, h, w, bias, act=act)
 
 
+class Scale(Part):
+    factor: torch.Tensor | None = None       # [width] float32, set by bind
+
+
 class PositionEncoding(Part):
     def embedding_table(self) -> torch.Tensor | None:
         """A [max_positions, width] table added to the token embedding, or None."""
@@ -143,6 +149,10 @@ class PositionEncoding(Part):
 
 
 class Embedding(Part):
+    # A part that sets ``keeps_output`` leaves a copy of its output in ``keep`` (float32, shaped
+    # like x) itself when the model asks for one.
+    keeps_output = False
+
     def forward(self, ctx, x, position: PositionEncoding) -> None:
         raise NotImplementedError
 
@@ -153,7 +163,8 @@ class Head(Part):
 
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Part]]] = {
-    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "embedding": {}, "head": {},
+    "mixer": {}, "feed_forward": {}, "norm": {}, "scale": {}, "position": {}, "embedding": {},
+    "head": {},
 }
 
 
@@ -174,6 +185,10 @@ def register_feed_forward(kind, factory, *, replace=False):
 
 def register_norm(kind, factory, *, replace=False):
     _register("norm", kind, factory, replace)
+
+
+def register_scale(kind, factory, *, replace=False):
+    _register("scale", kind, factory, replace)
 
 
 def register_position(kind, factory, *, replace=False):

@@ -6,13 +6,17 @@ numbers) and one rotated key part ``kr`` (``rot_dim`` numbers).  Head ``h`` has 
 ``q_plain . (W_uk[h] c) = (W_uk[h]^T q_plain) . c``, the kernels work on the latent directly:
 
     qa[h]  = W_uk[h]^T q_plain[h]                       (absorbed query, kv_rank numbers)
-    score  = (qa[h] . c_j + q_rot[h] . kr_j) * scale    over j <= i
-    weight = softmax over the scores and one sink logit per head (no key, no value)
+    score  = (qa[h] . c_j + q_rot[h] . kr_j) * scale    over j <= i (``window``: i - j < window)
+    weight = softmax over the scores (``sink``: and one sink logit per head, no key, no value)
     out[h] = W_uv[h] (sum_j weight_j c_j)
 
 Rotary positions act on interleaved pairs of the rotated parts.  A layer built with
 ``shares_cache`` has no latent projection: it reads the rows another layer call wrote (the
 schedule names the entry) with its own queries, expansions and sink.
+
+With ``q_down`` the queries come through a latent of their own: ``c_q = rms_norm(W_dq h)`` of
+``q_rank`` numbers, formed in the launch that writes the cache row (both latents are columns of
+one input projection), and the query matrix maps c_q instead of h.
 """
 
 from __future__ import annotations
@@ -26,29 +30,43 @@ class LatentAttention(Mixer):
     def __init__(self, *, width: int, n_heads: int, dim: int, rot_dim: int, vdim: int,
                  kv_rank: int, scale: float, rot_base: float, rot_dims: int, eps: float,
                  q_weight: str, latent_weight: str | None, latent_norm: str | None,
-                 key_up: str, value_up: str, sink: str, out_weight: str,
-                 shares_cache: bool = False):
+                 key_up: str, value_up: str, sink: str | None, out_weight: str,
+                 shares_cache: bool = False, window: int = 0, q_down: str | None = None,
+                 q_down_norm: str | None = None, q_rank: int = 0):
         if rot_dims % 2 or not 0 <= rot_dims <= rot_dim:
             raise ValueError(f"rot_dims must be even and at most rot_dim, got {rot_dims}")
         if shares_cache == (latent_weight is not None):
             raise ValueError("a layer either projects its own latent or shares another's")
+        if (q_down is None) != (q_down_norm is None) or (q_down is None) != (q_rank == 0):
+            raise ValueError("a query latent has a matrix, a norm and a size")
+        if q_down is not None and shares_cache:
+            raise ValueError("a layer that shares a latent projects its queries directly")
+        if window < 0:
+            raise ValueError("a window is not negative")
+        self.window, self.q_rank = int(window), int(q_rank)
         self.width, self.H, self.D, self.P, self.V, self.R = (width, n_heads, dim, rot_dim, vdim,
                                                               kv_rank)
         self.scale = float(torch.tensor(float(scale), dtype=torch.float64).to(torch.float32))
         self.rot_base, self.rot_dims, self.eps = float(rot_base), int(rot_dims), float(eps)
         self.names = dict(q=q_weight, dkv=latent_weight, dkv_norm=latent_norm, uk=key_up,
-                          uv=value_up, sink=sink, o=out_weight)
+                          uv=value_up, sink=sink, o=out_weight, dq=q_down, dq_norm=q_down_norm)
         self.shares_cache = bool(shares_cache)
         self.q_width = self.H * (self.D + self.P)
-        self.in_width = self.q_width + (0 if shares_cache else self.R + self.P)
+        # columns of the input projection: the queries or their latent, then the key/value latent
+        self.head_width = self.q_rank or self.q_width
+        self.in_width = self.head_width + (0 if shares_cache else self.R + self.P)
 
     def tensor_requests(self):
         n = self.names
-        req = {n["q"]: TensorRequest((self.q_width, self.width), "matrix"),
+        req = {n["q"]: TensorRequest((self.q_width, self.q_rank or self.width), "matrix"),
                n["uk"]: TensorRequest((self.H * self.D, self.R), "matrix"),
                n["uv"]: TensorRequest((self.H * self.V, self.R), "matrix"),
-               n["sink"]: TensorRequest((self.H,), "vector"),
                n["o"]: TensorRequest((self.width, self.H * self.V), "matrix")}
+        if n["sink"]:
+            req[n["sink"]] = TensorRequest((self.H,), "vector")
+        if n["dq"]:
+            req[n["dq"]] = TensorRequest((self.q_rank, self.width), "matrix")
+            req[n["dq_norm"]] = TensorRequest((self.q_rank,), "vector")
         if not self.shares_cache:
             req[n["dkv"]] = TensorRequest((self.R + self.P, self.width), "matrix")
             req[n["dkv_norm"]] = TensorRequest((self.R,), "vector")
@@ -57,9 +75,12 @@ class LatentAttention(Mixer):
     def bind(self, tensors):
         n = self.names
         wq = tensors[n["q"]]
-        # one input projection: the queries, then (for a layer with a latent of its own) the
-        # latent and the shared key part
-        self.w_in = wq if self.shares_cache else torch.cat([wq, tensors[n["dkv"]]]).contiguous()
+        # one input projection: the queries (or the latent they come through), then (for a layer
+        # with a latent of its own) the latent and the shared key part
+        first = tensors[n["dq"]] if n["dq"] else wq
+        self.w_in = first if self.shares_cache else torch.cat([first, tensors[n["dkv"]]]).contiguous()
+        self.w_q_up = wq if n["dq"] else None
+        self.q_norm_w = tensors[n["dq_norm"]] if n["dq"] else None
         self.norm_w = None if self.shares_cache else tensors[n["dkv_norm"]]
         # k-major per head: [H, D, R] maps q_plain to the latent, [H, R, V] maps it to a value
         self.w_absorb = tensors[n["uk"]].view(self.H, self.D, self.R).contiguous()
@@ -69,7 +90,7 @@ class LatentAttention(Mixer):
         if wq.dtype == torch.bfloat16:
             self.w_absorb_nk = self.w_absorb.transpose(1, 2).contiguous()
             self.w_expand_nk = tensors[n["uv"]].view(self.H, self.V, self.R).contiguous()
-        self.sink = tensors[n["sink"]]
+        self.sink = tensors[n["sink"]] if n["sink"] else None
         self.w_out = tensors[n["o"]]
         i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
         freq = torch.pow(torch.tensor(self.rot_base, dtype=torch.float64),
@@ -77,9 +98,11 @@ class LatentAttention(Mixer):
         self.freq = freq.to(torch.float32).to(wq.device)
 
     def cache_request(self):
-        return CacheRequest(kv_heads=1, head_dim=self.R + self.P, window=0, planes=1)
+        return CacheRequest(kv_heads=1, head_dim=self.R + self.P, window=self.window, planes=1)
 
-    def forward(self, ctx, h, x, cache):
+    writes_fresh = True
+
+    def forward(self, ctx, h, x, cache, fresh=False):
         ops, T = ctx.ops, h.shape[0]
         H, D, P, V, R = self.H, self.D, self.P, self.V, self.R
         proj = ctx.buffer("latent_proj", (T, self.in_width), torch.float32)
@@ -90,20 +113,30 @@ class LatentAttention(Mixer):
         if cache.writes:
             if self.shares_cache:
                 raise RuntimeError("a layer that shares a latent cache cannot write it")
+            more = dict(rot)
+            if self.q_rank:                      # the query latent's norm rides along
+                cq = ctx.buffer("latent_cq", (T, self.q_rank), ctx.dtype)
+                more.update(q_out=cq, q_norm=self.q_norm_w)
             ops.latent_append(cache.pool, proj, self.norm_w, cache.table, ctx.tok_pos,
-                              ctx.tok_req, c_offset=self.q_width, rank=R, rot_dim=P,
-                              eps=self.eps, page_size=cache.page_size, status=ctx.status, **rot)
+                              ctx.tok_req, c_offset=self.head_width, rank=R, rot_dim=P,
+                              eps=self.eps, page_size=cache.page_size, status=ctx.status, **more)
+        q = proj
+        if self.q_rank:
+            q = ctx.buffer("latent_q", (T, self.q_width), torch.float32)
+            ops.linear(q, cq, self.w_q_up)
         qa = ctx.buffer("latent_qa", (T, H * R), torch.float32)
-        ops.grouped_linear(qa, proj, self.w_absorb, a_offset=0, a_group_stride=D + P,
+        ops.grouped_linear(qa, q, self.w_absorb, a_offset=0, a_group_stride=D + P,
                            w_nk=self.w_absorb_nk)
         lat = ctx.buffer("latent_mix", (T, H * R), torch.float32)
-        ops.latent_attention(lat, qa, proj, cache.pool, cache.table, ctx.tok_pos, ctx.tok_req,
+        if self.window:
+            rot["window"] = self.window
+        ops.latent_attention(lat, qa, q, cache.pool, cache.table, ctx.tok_pos, ctx.tok_req,
                              self.sink, n_heads=H, rank=R, rot_dim=P, qr_head_stride=D + P,
                              qr_offset=D, scale=self.scale, page_size=cache.page_size,
                              status=ctx.status, plan=ctx.plan, **rot)
         att = ctx.buffer("latent_heads", (T, H * V), ctx.dtype)
         ops.grouped_linear(att, lat, self.w_expand, w_nk=self.w_expand_nk)
-        ops.linear(x, att, self.w_out, None, residual=x)
+        ops.linear(x, att, self.w_out, None, residual=None if fresh else x)
 
 
 register_mixer("latent_attention", LatentAttention)

@@ -207,10 +207,56 @@ class SandwichNormBlock(Block):
                 self.side.forward(ctx, h, x, **extra)
 
 
+class ScaledParallelBlock(Block):
+    """A parallel block whose sublayers' outputs are scaled column by column:
+
+        h = norm1(x);  x += scale1 * mixer(h) + scale2 * feed_forward(h)
+
+    Each sublayer writes a float32 block of its own, and one launch adds both into the stream.
+    That launch also adds the embedding's output when the schedule wants it before the call that
+    runs next, and forms the rows of the next block's norm when that block is of this arrangement
+    and its norm is a layer norm (``ctx.normed_ahead``).  A layer may leave ``feed_forward`` and
+    ``scale2`` out (both or neither)."""
+
+    slots = {"norm1": "norm", "mixer": "mixer", "scale1": "scale", "feed_forward": "feed_forward",
+             "scale2": "scale"}
+    optional = ("feed_forward", "scale2")
+    takes_norm_ahead = True
+
+    def __init__(self, spec: LayerSpec):
+        super().__init__(spec)
+        if (self.feed_forward is None) != (self.scale2 is None):
+            raise ValueError("arrangement 'scaled_parallel': feed_forward and scale2 come together")
+
+    def forward(self, ctx, x, cache):
+        T, W = x.shape
+        h = ctx.buffer("normed", (T, W), ctx.dtype)
+        if not ctx.normed_ahead:
+            self.norm1.forward(ctx, h, x)
+        y1 = ctx.buffer("mixer_out", (T, W), torch.float32)
+        y1 = OutputNormBlock._run(self.mixer, ctx, h, y1, cache)
+        more = {}
+        if self.feed_forward is not None:
+            y2 = ctx.buffer("feed_forward_out", (T, W), torch.float32)
+            more.update(y2=OutputNormBlock._run(self.feed_forward, ctx, h, y2),
+                        s2=self.scale2.factor)
+        if ctx.next_adds_embedding:
+            more["again"] = ctx.embedding_output
+        ahead = None
+        if getattr(ctx.next_block, "takes_norm_ahead", False):
+            ahead = getattr(ctx.next_block.norm1, "row_norm", None)
+        if ahead is not None:
+            more.update(out=h, norm=ahead())
+        ctx.ops.residual_mix(x, y1, self.scale1.factor, **more)
+        ctx.normed_ahead = ahead is not None
+        ctx.embedding_added = ctx.next_adds_embedding
+
+
 _ARRANGEMENTS: dict[str, Callable[[LayerSpec], Block]] = {"pre_norm": PreNormBlock,
                                                           "parallel": ParallelBlock,
                                                           "output_norm": OutputNormBlock,
-                                                          "sandwich_norm": SandwichNormBlock}
+                                                          "sandwich_norm": SandwichNormBlock,
+                                                          "scaled_parallel": ScaledParallelBlock}
 
 
 def register_arrangement(name: str, factory: Callable[[LayerSpec], Block], *, replace=False):
@@ -247,6 +293,7 @@ class Model:
         self.final_norm = build_part("norm", spec.final_norm)
         self.head = build_part("head", spec.head)
         self.schedule: tuple[LayerCall, ...] = spec.resolved_schedule()
+        self.keeps_embedding = any(call.adds_embedding for call in self.schedule)
         self.capturable = all(part.capturable for part in self.parts())
         self._derive_cache()
         self.dtype = None
@@ -358,15 +405,33 @@ class Model:
         T = ctx.n_rows
         x = ctx.buffer("residual", (T, spec.width), torch.float32)
         ctx.position = self.position          # mixers ask it whether it acts on queries and keys
-        self.embedding.forward(ctx, x, self.position)
         ctx.stream_copy_fresh = False         # no copy of the stream in the compute type yet
         ctx.normed_ahead = False              # nobody has formed the next block's first norm
+        ctx.embedding_added = False           # nobody has added what a call wants added before it
+        ctx.embedding_output = None
+        first = self.schedule[0] if self.schedule else None
+        ctx.next_block = self.blocks[first.layer] if first is not None else None
+        if self.keeps_embedding:              # kept aside: later calls add it to the stream again
+            keep = ctx.embedding_output = ctx.buffer("embedding_output", (T, spec.width),
+                                                     torch.float32)
+            if self.embedding.keeps_output:
+                self.embedding.forward(ctx, x, self.position, keep=keep)
+            else:
+                self.embedding.forward(ctx, x, self.position)
+                keep.copy_(x)
+        else:
+            self.embedding.forward(ctx, x, self.position)
         for idx, call in enumerate(self.schedule):
             ctx.call_index = idx
+            if call.adds_embedding and not ctx.embedding_added:
+                ctx.ops.residual_mix(x, again=ctx.embedding_output)
+                ctx.stream_copy_fresh = ctx.normed_ahead = False
+            ctx.embedding_added = False
             cache = ctx.cache_view(call) if call.cache in self.entry_location else None
             block = self.blocks[call.layer]
-            ctx.next_block = (self.blocks[self.schedule[idx + 1].layer]
-                              if idx + 1 < len(self.schedule) else None)
+            nxt = self.schedule[idx + 1] if idx + 1 < len(self.schedule) else None
+            ctx.next_block = self.blocks[nxt.layer] if nxt is not None else None
+            ctx.next_adds_embedding = nxt is not None and nxt.adds_embedding
             block.forward(ctx, x, cache)
             if not getattr(block, "keeps_stream_copy", False):
                 ctx.stream_copy_fresh = False

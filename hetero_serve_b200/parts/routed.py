@@ -21,6 +21,11 @@ experts and is added to their sum.
 A third rule (``scoring="table"``) has no router: an integer table [vocab, top] names the
 experts of every token id, each weighing 1/top; and a third expert (``activation="relu2"``) has
 no gate matrix: y = relu(W_up h)^2.
+
+A fourth rule (``scoring="softmax_corrected"``): s = softmax(W_r h) in float32 over all outputs of
+the router; the ``top`` largest of s + correction are chosen (the lower index wins a tie) and
+weigh s * ``weight_scale``, neither corrected nor renormalised.  With ``identity`` the router has
+that many outputs behind the experts': choosing one adds weight * h itself (no tensors).
 """
 
 from __future__ import annotations
@@ -29,7 +34,7 @@ import torch
 
 from .base import FeedForward, TensorRequest, build_part, register_feed_forward
 
-SCORINGS = ("sigmoid_groups", "softmax_top", "table")
+SCORINGS = ("sigmoid_groups", "softmax_top", "table", "softmax_corrected")
 
 
 class RoutedExperts(FeedForward):
@@ -38,7 +43,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, *, width: int, ff: int, experts: int, top: int, router: str,
                  expert_prefix: str, groups: int = 1, keep: int = 1, limit: float = 0.0,
                  scoring: str = "sigmoid_groups", activation: str = "clamped",
-                 router_bias: str | None = None, shared=None, table_rows: int = 0):
+                 router_bias: str | None = None, shared=None, table_rows: int = 0,
+                 correction: str | None = None, weight_scale: float = 1.0, identity: int = 0):
         if scoring not in SCORINGS:
             raise ValueError(f"unknown scoring {scoring!r}; known: {SCORINGS}")
         if activation not in ("clamped", "silu", "relu2"):
@@ -50,10 +56,20 @@ class RoutedExperts(FeedForward):
                 raise ValueError("top experts must fit into the kept groups")
             if router_bias is not None:
                 raise ValueError("the grouped sigmoid rule takes no router bias")
-        elif not 0 < top <= experts:
+        elif not 0 < top <= experts + identity:
             raise ValueError(f"{top} chosen experts of {experts}")
         if scoring == "table" and (table_rows <= 0 or router_bias is not None):
             raise ValueError("the table rule needs the table's rows and takes no router bias")
+        if scoring != "softmax_corrected" and (correction is not None or identity
+                                               or weight_scale != 1.0):
+            raise ValueError("correction, weight_scale and identity belong to 'softmax_corrected'")
+        if scoring == "softmax_corrected" and router_bias is not None:
+            raise ValueError("the corrected softmax rule takes no router bias")
+        if identity < 0:
+            raise ValueError(f"{identity} identity experts")
+        self.correction_name, self.weight_scale = correction, float(weight_scale)
+        self.identity = int(identity)
+        self.outputs = experts + self.identity         # of the router
         self.table_rows = int(table_rows)
         self.width, self.ff, self.E, self.top = width, ff, experts, top
         self.groups, self.keep, self.limit = groups, keep, float(limit)
@@ -71,9 +87,11 @@ class RoutedExperts(FeedForward):
         if self.scoring == "table":
             req = {self.router_name: TensorRequest((self.table_rows, self.top), "int")}
         else:
-            req = {self.router_name: TensorRequest((self.E, self.width), "float32")}
+            req = {self.router_name: TensorRequest((self.outputs, self.width), "float32")}
         if self.bias_name:
             req[self.bias_name] = TensorRequest((self.E,), "vector")
+        if self.correction_name:
+            req[self.correction_name] = TensorRequest((self.outputs,), "vector")
         if self.shared is not None:
             req.update(self.shared.tensor_requests())
         for e in range(self.E):
@@ -86,6 +104,7 @@ class RoutedExperts(FeedForward):
     def bind(self, tensors):
         self.w_router = tensors[self.router_name]
         self.b_router = tensors[self.bias_name] if self.bias_name else None
+        self.correction = tensors[self.correction_name] if self.correction_name else None
         if self.shared is not None:
             self.shared.bind({n: tensors[n] for n in self.shared.tensor_requests()})
         # prompt portions in bfloat16 form the logits as one product on the tensor cores (exact
@@ -112,13 +131,11 @@ class RoutedExperts(FeedForward):
                 if fresh:
                     x.zero_()
                 self.shared.forward(ctx, h, x)
-        elif fresh:
-            x.zero_()
         idx = ctx.buffer("route_idx", (T, self.top), torch.int32)
         wts = ctx.buffer("route_w", (T, self.top), torch.float32)
         z = None
         if self.w_router_lp is not None and T >= 64:
-            z = ctx.buffer("route_z", (T, self.E), torch.float32)
+            z = ctx.buffer("route_z", (T, self.outputs), torch.float32)
             ops.linear(z, h, self.w_router_lp)
         if self.scoring == "table":
             ops.moe_route_table(idx, wts, self.w_router, ctx.tok_ids, ctx.tok_req, top=self.top,
@@ -126,11 +143,18 @@ class RoutedExperts(FeedForward):
         elif self.scoring == "softmax_top":
             ops.moe_route_top(idx, wts, h, self.w_router, self.b_router, ctx.tok_req,
                               top=self.top, z=z)
+        elif self.scoring == "softmax_corrected":
+            ops.moe_route_softmax(idx, wts, h, self.w_router, self.correction, ctx.tok_req,
+                                  top=self.top, scale=self.weight_scale, z=z)
         else:
             ops.moe_route(idx, wts, h, self.w_router, ctx.tok_req, top=self.top,
                           n_groups=self.groups, keep=self.keep, z=z)
         y = ctx.buffer("expert_act", (T * self.top, self.ff), torch.float32)
         more = {"act": self.activation} if self.activation != "clamped" else {}
+        if self.identity:
+            more["identity"] = self.identity
+        if fresh and self.shared is None:          # nothing else has opened x: write, do not add
+            more["fresh"] = True
         ops.moe_experts(x, y, h, self.w_gate, self.w_up, self.w_down, idx, wts, ctx.tok_req,
                         limit=self.limit, **more)
 

@@ -16,7 +16,7 @@ cache entry; ``writes_cache=False`` makes the call a reader only).
 
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from types import MappingProxyType
 from typing import Any, Mapping
 
@@ -82,6 +82,7 @@ class LayerCall:
     layer: int                    # index into ModelSpec.layers
     cache: int | None = None      # cache entry this call uses; None → one of its own
     writes_cache: bool = True     # False: only reads what an earlier call wrote
+    adds_embedding: bool = False  # the embedding's output is added to the stream before the call
 
 
 @dataclass(frozen=True)
@@ -113,7 +114,7 @@ class ModelSpec:
                 while nxt in used:
                     nxt += 1
                 used.add(nxt)
-                out.append(LayerCall(call.layer, nxt, call.writes_cache))
+                out.append(replace(call, cache=nxt))
             else:
                 out.append(call)
         # entries must be numbered densely so they can index a pool

@@ -93,6 +93,10 @@ class LayerNorm(Norm):
         self.weight = tensors[self.wn]
         self.bias = tensors[self.bn] if self.bn else torch.zeros_like(self.weight)
 
+    def row_norm(self):
+        """(weight, bias, eps) for a launch that forms this norm of rows it has at hand."""
+        return self.weight, self.bias if self.bn else None, self.eps
+
     def add_normed(self, ctx, x, y, h=None, then=None):
         """x += norm(y) for a float32 block ``y``.  With ``then=(norm, out)``, ``out`` also
         receives ``norm(x)`` of the new rows (another layer norm's output, for the sublayer

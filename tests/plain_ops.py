@@ -184,10 +184,15 @@ class PlainOps:
         return out
 
     def latent_append(self, pool, proj, norm_w, table, tok_pos, tok_req, *, c_offset, rank,
-                      rot_dim, eps, page_size, status, freq=None, rot_dims=0):
+                      rot_dim, eps, page_size, status, freq=None, rot_dims=0, q_out=None,
+                      q_norm=None, q_offset=0):
         rows = pool.view(-1, page_size, rank + rot_dim)
         for t in range(proj.shape[0]):
             r = int(tok_req[t])
+            if q_out is not None:
+                q = proj[t, q_offset:q_offset + q_out.shape[1]].to(self.cd)
+                q_out[t] = 0 if r < 0 else (q / torch.sqrt((q * q).mean() + eps)
+                                            * q_norm.to(self.cd)).to(q_out.dtype)
             if r < 0:
                 continue
             p = int(tok_pos[t])
@@ -200,7 +205,7 @@ class PlainOps:
 
     def latent_attention(self, out, qa, qr, pool, table, tok_pos, tok_req, sink, *, n_heads,
                          rank, rot_dim, qr_head_stride, qr_offset, scale, page_size, status,
-                         freq=None, rot_dims=0, plan=None):
+                         freq=None, rot_dims=0, plan=None, window=0):
         rows = pool.view(-1, page_size, rank + rot_dim)
         scale32 = float(torch.tensor(scale, dtype=torch.float32))
         for t in range(out.shape[0]):
@@ -209,13 +214,16 @@ class PlainOps:
                 out[t] = 0
                 continue
             p = int(tok_pos[t])
-            js = torch.arange(0, p + 1)
+            js = torch.arange(max(0, p + 1 - window) if window else 0, p + 1)
             keys = rows[table[r, js // page_size].long(), js % page_size].to(self.cd)
             c, kr = keys[:, :rank], keys[:, rank:]
             for h in range(n_heads):
                 qh = qa[t, h * rank:(h + 1) * rank].to(self.cd)
                 lo = qr_offset + h * qr_head_stride
                 s = (c @ qh + kr @ self._turned(qr[t, lo:lo + rot_dim], p, freq, rot_dims)) * scale32
+                if sink is None:
+                    out[t, h * rank:(h + 1) * rank] = (torch.softmax(s, 0) @ c).to(out.dtype)
+                    continue
                 top = torch.maximum(s.max(), sink[h].to(self.cd))
                 e = torch.exp(s - top)
                 den = e.sum() + torch.exp(sink[h].to(self.cd) - top)
@@ -305,8 +313,21 @@ class PlainOps:
             sel_w[t] = (s[idx] / (s[idx].sum() + 1e-20)).to(sel_w.dtype)
 
     def moe_experts(self, x, y, h, w_gate, w_up, w_down, sel_idx, sel_w, tok_req, *, limit,
-                    act="clamped"):
+                    act="clamped", identity=0, fresh=False):
         T, top = sel_idx.shape
+        if fresh:
+            live = tok_req[:T] >= 0
+            x[:T][live] = 0
+        if identity:
+            E = w_up.shape[0]
+            behind = (sel_idx >= E) & (sel_idx < E + identity)
+            for t in range(T):
+                if int(tok_req[t]) >= 0:
+                    share = (sel_w[t] * behind[t]).to(self.cd).sum()
+                    x[t] = (x[t].to(self.cd) + share * h[t].to(self.cd)).to(x.dtype)
+            # what is left has a weight of 0 on some expert with matrices
+            sel_w = torch.where(sel_idx >= E, torch.zeros_like(sel_w), sel_w)
+            sel_idx = torch.where(sel_idx >= E, torch.zeros_like(sel_idx), sel_idx)
         if act == "relu2":
             for t in range(T):
                 if int(tok_req[t]) < 0:
@@ -356,6 +377,45 @@ class PlainOps:
             idx = torch.tensor(order)
             sel_idx[t] = idx.to(torch.int32)
             sel_w[t] = torch.softmax(logits[idx], 0).to(sel_w.dtype)
+
+    def moe_route_softmax(self, sel_idx, sel_w, h, w_router, correction, tok_req, *, top, scale,
+                          z=None):
+        for t in range(sel_idx.shape[0]):
+            if int(tok_req[t]) < 0:
+                continue
+            logits = (w_router.to(self.cd) @ h[t].to(self.cd)) if z is None else z[t].to(self.cd)
+            s = torch.softmax(logits, 0)
+            c = s if correction is None else s + correction.to(self.cd)
+            idx = torch.tensor(sorted(range(s.shape[0]), key=lambda e: (-float(c[e]), e))[:top])
+            sel_idx[t] = idx.to(torch.int32)
+            sel_w[t] = (s[idx] * scale).to(sel_w.dtype)
+
+    # -- the stream around a parallel block ---------------------------------------------------
+    def _ln_or(self, v, g, b, eps):
+        return self._ln(v, g, torch.zeros_like(g) if b is None else b, eps)
+
+    def embed_norm(self, x, ids, req, table, weight, bias, eps, status, feedback=None, keep=None,
+                   out=None, norm=None):
+        live = (req[:x.shape[0]] >= 0)[:, None]
+        tok = torch.tensor([max(0, self._token(ids, t, feedback)) for t in range(x.shape[0])])
+        row = self._ln_or(table[tok].to(self.cd), weight, bias, eps)
+        x.copy_(torch.where(live, row, torch.zeros_like(row)).to(x.dtype))
+        if keep is not None:
+            keep.copy_(x)
+        if out is not None:
+            v = self._ln_or(x.to(self.cd), *norm)
+            out.copy_(torch.where(live, v, torch.zeros_like(v)).to(out.dtype))
+
+    def residual_mix(self, x, y1=None, s1=None, y2=None, s2=None, again=None, out=None, norm=None):
+        v = x.to(self.cd)
+        for y, s in ((y1, s1), (y2, s2)):
+            if y is not None:
+                v = v + y.to(self.cd) * s.to(self.cd)
+        if again is not None:
+            v = v + again.to(self.cd)
+        x.copy_(v.to(x.dtype))
+        if out is not None:
+            out.copy_(self._ln_or(x.to(self.cd), *norm).to(out.dtype))
 
     def gated_act(self, out, gu, h=None, w_s=None, tok_req=None, act="silu"):
         ff = out.shape[1]
