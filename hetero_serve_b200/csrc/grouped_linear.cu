@@ -7,10 +7,16 @@
 // transposed once at binding) so that a warp's loads of one k are contiguous.  A block covers TT
 // tokens x 32 output columns; its four warps each sum a quarter of k for every column, and the
 // quarters are added in a fixed order, so a row's result depends on nothing else in the batch.
+//
+// `list` (may be null): a step's attention plan; then row i of the launch is the i-th single-query
+// token of the plan (`n_tokens` bounds their number) and no other token is touched.
 #include "common.cuh"
 #include "mma_tiles.cuh"
 
 namespace hs {
+
+// the token of row i: list = {count, -, -, -, token, -, -, token, ...}
+__device__ __forceinline__ int gl_token(const int* list, int i) { return list ? list[4 + 3 * i] : i; }
 
 constexpr int GL_TT = 8;          // tokens a block covers
 constexpr int GL_THREADS = 128;   // four warps: each takes a quarter of the summed index
@@ -20,19 +26,23 @@ template <typename TW, typename TO>
 __global__ void __launch_bounds__(GL_THREADS)
 grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
                       const TW* __restrict__ w, int n_tokens, int a_stride, int a_off,
-                      int a_gstride, int groups, int n, int k) {
+                      int a_gstride, int groups, int n, int k, const int* __restrict__ list) {
   extern __shared__ float s_a[];                    // [GL_TT][k]
   pdl_trigger();
   pdl_wait();
   __shared__ float s_part[GL_THREADS / 32][GL_TT][GL_COLS];
   const int t0 = blockIdx.x * GL_TT;
+  if (list) n_tokens = min(n_tokens, list[0]);
+  if (t0 >= n_tokens) return;
   const int g = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int j = blockIdx.z * GL_COLS + lane;
   const int nt = min(GL_TT, n_tokens - t0);
   for (int i = threadIdx.x; i < GL_TT * k; i += GL_THREADS) {
     const int tt = i / k, kk = i - tt * k;
-    s_a[i] = tt < nt ? a[(size_t)(t0 + tt) * a_stride + a_off + (size_t)g * a_gstride + kk] : 0.f;
+    s_a[i] = tt < nt ? a[(size_t)gl_token(list, t0 + tt) * a_stride + a_off +
+                         (size_t)g * a_gstride + kk]
+                     : 0.f;
   }
   __syncthreads();
   float acc[GL_TT];
@@ -58,7 +68,7 @@ grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
     const int col = blockIdx.z * GL_COLS + c;
     if (tt < nt && col < n) {
       const float v = ((s_part[0][tt][c] + s_part[1][tt][c]) + s_part[2][tt][c]) + s_part[3][tt][c];
-      out[(size_t)(t0 + tt) * groups * n + (size_t)g * n + col] = from_f<TO>(v);
+      out[(size_t)gl_token(list, t0 + tt) * groups * n + (size_t)g * n + col] = from_f<TO>(v);
     }
   }
 }
@@ -76,17 +86,20 @@ template <typename TO, int SPLIT>
 __global__ void __launch_bounds__(128)
 grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
                           const __nv_bfloat16* __restrict__ w, int n_tokens, int a_stride,
-                          int a_off, int a_gstride, int groups, int N, int K, int vec) {
+                          int a_off, int a_gstride, int groups, int N, int K, int vec,
+                          const int* __restrict__ list) {
   __shared__ __align__(16) __nv_bfloat16 s_a[2][SPLIT][TM * TS];
   __shared__ __align__(16) __nv_bfloat16 s_b[2][TN * TS];
   pdl_trigger();
   pdl_wait();
   const int t0 = blockIdx.x * TM, n0 = blockIdx.y * TN, g = blockIdx.z;
+  if (list) n_tokens = min(n_tokens, list[0]);
+  if (t0 >= n_tokens) return;
   const int rows = min(TM, n_tokens - t0), ncols = min(TN, N - n0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int wm = (warp >> 1) * 32, wn = (warp & 1) * 32;
   const int gq = lane >> 2, tq = lane & 3;
-  const float* a_base = a + (size_t)t0 * a_stride + a_off + (size_t)g * a_gstride;
+  const float* a_base = a + a_off + (size_t)g * a_gstride;
   const __nv_bfloat16* b_base = w + ((size_t)g * N + n0) * K;
   auto b_row = [&](int r) { return b_base + (size_t)r * K; };
   float ra[2][8];
@@ -95,7 +108,8 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
     for (int j = 0; j < 2; ++j) {
       const int c = threadIdx.x + 128 * j;
       const int r = c >> 2, col = (c & 3) * 8;
-      const float* src = a_base + (size_t)r * a_stride + k0 + col;
+      const float* src = a_base + k0 + col;
+      if (r < rows) src += (size_t)gl_token(list, t0 + r) * a_stride;
       if (r >= rows) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) ra[j][i] = 0.f;
@@ -189,7 +203,7 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
         for (int q = 0; q < 2; ++q) {
           const int c = wn + 8 * j + 2 * tq + q;
           if (c < ncols)
-            out[(size_t)(t0 + r) * groups * N + (size_t)g * N + n0 + c] =
+            out[(size_t)gl_token(list, t0 + r) * groups * N + (size_t)g * N + n0 + c] =
                 from_f<TO>(acc[i][j][2 * half + q]);
         }
       }
@@ -199,7 +213,7 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
 
 HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_tokens,
                                 int a_stride, int a_off, int a_gstride, int groups, int n, int k,
-                                int w_dtype, int out_dtype, void* stream) {
+                                int w_dtype, int out_dtype, const int* list, void* stream) {
   if (!out || !a || !w) return HS_ERR_ARGUMENT;
   if (groups <= 0 || n <= 0 || k <= 0) return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
@@ -214,7 +228,7 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
     if (smem > 48 * 1024)                                                                     \
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     e = hs_launch(kern, grid, dim3(hs::GL_THREADS), smem, st, hs_pdl_enabled(), (TO*)out, a, \
-                  (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k);          \
+                  (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, list);    \
   } while (0)
   if (w_dtype == HS_DT_F32 && out_dtype == HS_DT_F32) HS_GL(float, float);
   else if (w_dtype == HS_DT_BF16 && out_dtype == HS_DT_F32) HS_GL(__nv_bfloat16, float);
@@ -228,7 +242,8 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
 // HS_ERR_UNSUPPORTED for what it does not take (the caller then uses the kernel above).
 HS_EXPORT int hs_grouped_linear_mma(void* out, const float* a, const void* w_nk, int n_tokens,
                                     int a_stride, int a_off, int a_gstride, int groups, int n,
-                                    int k, int out_dtype, int split, void* stream) {
+                                    int k, int out_dtype, int split, const int* list,
+                                    void* stream) {
   if (!out || !a || !w_nk) return HS_ERR_ARGUMENT;
   if (groups <= 0 || n <= 0 || k <= 0 || k % hs::TK || (split != 1 && split != 3))
     return HS_ERR_UNSUPPORTED;
@@ -241,16 +256,16 @@ HS_EXPORT int hs_grouped_linear_mma(void* out, const float* a, const void* w_nk,
   cudaError_t e = cudaSuccess;
   if (out_dtype == HS_DT_F32 && split == 3)
     e = hs_launch(hs::grouped_linear_mma_kernel<float, 3>, grid, dim3(128), 0, st, pdl, (float*)out,
-                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec);
+                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec, list);
   else if (split == 3)
     return HS_ERR_UNSUPPORTED;
   else if (out_dtype == HS_DT_F32)
     e = hs_launch(hs::grouped_linear_mma_kernel<float, 1>, grid, dim3(128), 0, st, pdl, (float*)out,
-                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec);
+                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec, list);
   else if (out_dtype == HS_DT_BF16)
     e = hs_launch(hs::grouped_linear_mma_kernel<__nv_bfloat16, 1>, grid, dim3(128), 0, st, pdl,
                   (__nv_bfloat16*)out, a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k,
-                  vec);
+                  vec, list);
   else
     return HS_ERR_UNSUPPORTED;
   return e == cudaSuccess ? HS_OK : (int)e;

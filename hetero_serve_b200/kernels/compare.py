@@ -63,13 +63,23 @@ class TimedOps:
 
 
 _UNTIMED = {"stream", "register_kernel", "load_extension", "attention_plan_ints",
-            "plan_attention", "make_plan", "decode_wide", "decode_splits"}
+            "plan_attention", "make_plan", "decode_wide", "decode_splits",
+            "latent_prompt_rows"}
 
 
 def _contexts(batch):
     """Sum over the step's tokens of the keys each sees, and the distinct cache rows read."""
     seen = sum(n * start + n * (n + 1) // 2 for start, n in batch)
     rows = sum(start + n for start, n in batch)
+    return seen, rows
+
+
+def _windowed(batch, window):
+    """The same for queries that see the last ``window`` positions (0: all)."""
+    if window <= 0:
+        return _contexts(batch)
+    seen = sum(min(i + 1, window) for start, n in batch for i in range(start, start + n))
+    rows = sum(start + n - max(0, start + 1 - window) for start, n in batch)
     return seen, rows
 
 
@@ -99,8 +109,18 @@ def _flops_and_bytes(name, args, kw, batch):
             out, qa = args[:2]
             pool = args[3]
             H, R, P = kw["n_heads"], kw["rank"], kw["rot_dim"]
-            seen, rows = _contexts(batch)
+            seen, rows = _windowed(batch, kw.get("window", 0))
             return 2 * H * (2 * R + P) * seen, _nbytes(out, qa) + rows * (R + P) * pool.element_size()
+        if name == "latent_gather":
+            lat, rope, q_out, _base, q = args[:5]
+            _seen, rows = _windowed(batch, kw["window"])
+            return 0, rows * 2 * 2 * (lat.shape[1] + kw["rot_dim"]) + _nbytes(q_out, q)
+        if name == "latent_prompt_attention":
+            out, q, kv = args[:3]
+            H, D, P, V = kw["n_heads"], kw["dim"], kw["rot_dim"], kw["vdim"]
+            seen, rows = _windowed(batch, kw["window"])
+            return (2 * H * (D + P + V) * seen,
+                    _nbytes(out, q) + rows * 2 * (H * (D + V) + P))
         if name == "grouped_linear":
             out, a, w = args[:3]
             groups, k, n = w.shape
@@ -143,7 +163,20 @@ def _flops_and_bytes(name, args, kw, batch):
             live = len([1 for _s, n in batch if n > 0])
             cols = (2 * H * D + H * V) * 4
             return 5 * o.shape[0] * H * D * V, _nbytes(o) + o.shape[0] * cols + 2 * live * H * D * V * 4
-        if name in ("moe_route", "moe_route_top"):
+        if name == "latent_append":
+            pool, proj = args[:2]
+            q_out = kw.get("q_out")
+            cols = kw["rank"] + kw["rot_dim"]
+            read = cols + (q_out.shape[1] if q_out is not None else 0)
+            return 0, proj.shape[0] * (4 * read + cols * pool.element_size()) + _nbytes(q_out)
+        if name == "embed_norm":
+            x, table = args[0], args[3]
+            return 0, _nbytes(x, kw.get("keep"), kw.get("out")) + x.numel() * table.element_size()
+        if name == "residual_mix":
+            more = args[1:2] if len(args) > 1 else (kw.get("y1"),)
+            return 0, 2 * _nbytes(args[0]) + _nbytes(*more, kw.get("y2"), kw.get("again"),
+                                                     kw.get("out"))
+        if name in ("moe_route", "moe_route_top", "moe_route_softmax"):
             h, wr = args[2], args[3]
             return 2 * h.shape[0] * wr.shape[0] * wr.shape[1], _nbytes(h, wr)
         if name == "moe_experts":
@@ -228,8 +261,7 @@ def _flops_and_bytes(name, args, kw, batch):
                 last = start + n - 1
                 rows += last + 1 - max(0, start - win + 1) + max(0, (last - win + 1) // blk)
             return 2 * H * (D + V) * seen, _nbytes(out, q) + rows * G * (D + V) * pool.element_size()
-        if name in ("embed", "scale_", "rotary_pairs", "latent_append", "sample", "argmax",
-                    "kv_append"):
+        if name in ("embed", "scale_", "rotary_pairs", "sample", "argmax", "kv_append"):
             return 0, _nbytes(args[0])
     except Exception:                                   # an estimate must never stop a step
         pass

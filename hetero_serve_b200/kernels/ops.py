@@ -200,8 +200,11 @@ def _declare(lib) -> None:
         "hs_dyt_norm": [P, P, P, P, P, I, I, F, I, P],
         "hs_scale": [P, ctypes.c_longlong, F, P],
         "hs_rotary_pairs": [P, P, P, P, I, I, I, I, I, I, P],
-        "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P],
-        "hs_grouped_linear_mma": [P, P, P, I, I, I, I, I, I, I, I, I, P],
+        "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P, P],
+        "hs_grouped_linear_mma": [P, P, P, I, I, I, I, I, I, I, I, I, P, P],
+        "hs_latent_prefill_tc_takes": [I, I, I, I, I, F],
+        "hs_latent_gather": [P] * 11 + [I] * 12 + [P, I, P, P],
+        "hs_latent_prefill_tc": [P] * 6 + [I] * 10 + [F, P, P],
         "hs_latent_append": [P, P, P, P, P, P, I, I, I, I, I, F, I, I, I, I, P, P, I, P, P, I, I,
                              P],
         "hs_latent_attention": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, P, I,
@@ -339,6 +342,8 @@ class CudaOps:
         self.pdl = True            # programmatic dependent launch (see the property below)
         self._skinny_need: dict = {}
         self._moe_need: dict = {}
+        # windowed latent attention of prompt portions in expanded form, on tcgen05 tensor cores
+        self.latent_expanded = True
         self.latent_mma = True      # prompt portions of latent attention on the tensor cores
         self.biased_mma = True      # prompt portions of the biased chunk attention likewise
         self.pooled_mma = True      # ... and of the attention over a window and pooled blocks
@@ -1061,7 +1066,7 @@ class CudaOps:
                "rotary_pairs")
 
     def grouped_linear(self, out, a, w, *, a_offset=0, a_group_stride=None, w_nk=None,
-                       exact=False):
+                       exact=False, singles=None):
         """Block-diagonal linear: ``out[t, g*n + j] = sum_k a[t, a_offset + g*a_group_stride + k]
         * w[g, k, j]``.  ``a`` float32 (a group's input may be a slice of a wider row), ``w``
         [groups, k, n] (k-major), ``out`` [T, groups * n] float32 or of w's type.  ``w_nk`` is
@@ -1069,7 +1074,8 @@ class CudaOps:
         multiple of 32, the product runs on the tensor cores (``a`` rounded to bfloat16; with
         ``exact`` ``a`` enters as the sum of three bfloat16 terms, which loses nothing of a
         float32: for weights that are bfloat16 numbers the result is then the float32 product,
-        and ``out`` is float32)."""
+        and ``out`` is float32).  With ``singles`` (the step's attention plan) only the plan's
+        single-query tokens are worked on."""
         _want(a, "a", torch.float32, 2)
         _want(w, "w", _FLOATS, 3)
         _want(out, "out", _FLOATS, 2)
@@ -1082,19 +1088,24 @@ class CudaOps:
             raise KernelError("grouped_linear: the groups' inputs exceed a's row")
         if out.dtype != torch.float32 and out.dtype != w.dtype:
             raise KernelError("grouped_linear: out is float32 or of the weights' type")
+        listed = None
+        if singles is not None:
+            T, listed = min(T, singles.decode_cap), singles.data
+            if T == 0:
+                return
         self.launches += 1
         if (w_nk is not None and T >= 64 and w_nk.dtype == torch.bfloat16 and self.tensor_cores
                 and tuple(w_nk.shape) == (groups, n, k) and w_nk.is_contiguous()):
             code = self.lib.hs_grouped_linear_mma(_ptr(out), _ptr(a), _ptr(w_nk), T, a.shape[1],
                                                   int(a_offset), gs, groups, n, k,
                                                   _DT[out.dtype], 3 if exact else 1,
-                                                  self._stream())
+                                                  _ptr(listed), self._stream())
             if code != -1:
                 _check(code, f"grouped_linear_mma(groups={groups},n={n},k={k})")
                 return
         _check(self.lib.hs_grouped_linear(_ptr(out), _ptr(a), _ptr(w), T, a.shape[1],
                                           int(a_offset), gs, groups, n, k, _DT[w.dtype],
-                                          _DT[out.dtype], self._stream()),
+                                          _DT[out.dtype], _ptr(listed), self._stream()),
                f"grouped_linear(groups={groups},n={n},k={k})")
 
     # -- attention over a shared latent ---------------------------------------------------
@@ -1138,7 +1149,7 @@ class CudaOps:
 
     def latent_attention(self, out, qa, qr, pool, table, tok_pos, tok_req, sink, *, n_heads,
                          rank, rot_dim, qr_head_stride, qr_offset, scale, page_size, status,
-                         freq=None, rot_dims=0, plan=None, window=0):
+                         freq=None, rot_dims=0, plan=None, window=0, singles_only=False):
         """Causal softmax attention over cache rows ``[c (rank) | kr (rot_dim)]`` shared by all
         heads: score = (qa[t,h] . c + qr[t,h] . kr) * scale over every earlier position, or with
         ``window`` the last ``window`` ones (the token itself among them); with ``sink`` the
@@ -1148,7 +1159,8 @@ class CudaOps:
         unrotated and its first ``rot_dims`` entries are rotated as they are read.  With the
         step's ``plan`` and a bfloat16 cache, the plan's tiles (prompt portions) run on the
         tensor cores with the queries rounded to bfloat16, its single-query tokens on the CUDA
-        cores; without a plan every token runs on the CUDA cores."""
+        cores; without a plan every token runs on the CUDA cores.  With ``singles_only`` the
+        plan's tiles are left out (another operation serves them)."""
         _want(out, "out", torch.float32, 2)
         _want(qa, "qa", torch.float32, 2)
         _want(qr, "qr", torch.float32, 2)
@@ -1169,7 +1181,11 @@ class CudaOps:
         rot = int(rot_dims) if freq is not None else 0
         n_pages = pool.numel() // (page_size * W)
         listed = None
-        if (plan is not None and plan.tile_cap > 0 and pool.dtype == torch.bfloat16
+        if singles_only:
+            listed, n = plan.data, plan.decode_cap
+            if n == 0:
+                return
+        elif (plan is not None and plan.tile_cap > 0 and pool.dtype == torch.bfloat16
                 and self.tensor_cores and self.latent_mma):
             code = self.lib.hs_latent_prefill_mma(
                 _ptr(out), _ptr(qa), _ptr(qr), _ptr(pool), _ptr(table), _ptr(sink),
@@ -1205,6 +1221,76 @@ class CudaOps:
             table.shape[1], _DT[pool.dtype], _ptr(status), nsplit, _ptr(partial), _ptr(freq),
             rot, _ptr(listed), int(window), self._stream()),
             f"latent_attention(rank={rank},rot_dim={rot_dim})")
+
+    # -- prompt portions over a windowed latent: keys and values expanded per head -------------
+    LATENT_EXPANDED_BYTES = 1 << 31        # largest block of expanded rows a step may need
+
+    def latent_prompt_rows(self, plan, n_requests, *, n_heads, dim, rot_dim, vdim, rank, window,
+                           scale) -> int:
+        """Rows of the dense blocks with which the plan's prompt portions run in expanded form
+        (each portion's tokens and the window - 1 positions before them), or 0 when the kernels
+        do not take the sizes or the step has no portion."""
+        if (plan is None or plan.tile_cap <= 0 or window <= 0 or not self.tensor_cores
+                or not self.latent_expanded):
+            return 0
+        if not self.lib.hs_latent_prefill_tc_takes(int(dim), int(rot_dim), int(vdim), int(rank),
+                                                   int(window), float(scale)):
+            return 0
+        rows = plan.n_rows + min(n_requests, plan.tile_cap) * (window - 1)
+        return rows if 2 * rows * n_heads * (dim + vdim) <= self.LATENT_EXPANDED_BYTES else 0
+
+    def latent_gather(self, lat, rope, q_out, base, q, pool, table, req_start, req_len, tok_pos,
+                      tok_req, *, n_heads, dim, rank, rot_dim, window, page_size, status, freq=None,
+                      rot_dims=0):
+        """For every request that brings a prompt portion: the cache rows of the positions its
+        tokens see, dense (``lat`` [rows, rank], ``rope`` [rows, 64], padded with zeros; position
+        p of request r in row ``base[r] + p``), and its queries turned, rounded and padded
+        (``q_out`` [T, n_heads * (dim padded to 64 + 64)])."""
+        for t, nm in ((lat, "lat"), (rope, "rope"), (q_out, "q_out")):
+            _want(t, nm, torch.bfloat16, 2)
+        _want(pool, "pool", torch.bfloat16)
+        _want(q, "q", torch.float32, 2)
+        _want(base, "base", torch.int32, 1)
+        _want(table, "table", torch.int32, 2)
+        T, R = q_out.shape[0], base.shape[0]
+        W = rank + rot_dim
+        pad = -(-dim // 64) * 64
+        if lat.shape[1] != rank or tuple(rope.shape) != (lat.shape[0], 64) or rot_dim > 64 or \
+                q_out.shape[1] != n_heads * (pad + 64) or q.shape[0] < T or \
+                q.shape[1] != n_heads * (dim + rot_dim) or pool.numel() % (page_size * W):
+            raise KernelError("latent_gather: shapes do not fit")
+        if table.shape[0] < R or req_start.shape[0] < R or req_len.shape[0] < R or \
+                tok_pos.shape[0] < T or tok_req.shape[0] < T:
+            raise KernelError("latent_gather: the batch does not fit")
+        self.launches += 1
+        _check(self.lib.hs_latent_gather(
+            _ptr(lat), _ptr(rope), _ptr(q_out), _ptr(base), _ptr(q), _ptr(pool), _ptr(table),
+            _ptr(req_start), _ptr(req_len), _ptr(tok_pos), _ptr(tok_req), R, T, lat.shape[0],
+            int(window), DECODE_MAX_NEW, rank, rot_dim, n_heads, dim, page_size,
+            pool.numel() // (page_size * W), table.shape[1], _ptr(freq),
+            int(rot_dims) if freq is not None else 0, _ptr(status), self._stream()),
+            f"latent_gather(rank={rank},dim={dim})")
+
+    def latent_prompt_attention(self, out, q, kv, rope, base, plan, *, n_heads, dim, rot_dim, vdim,
+                                rank, window, scale, status):
+        """Softmax attention of the plan's prompt portions over the last ``window`` positions:
+        ``q`` as ``latent_gather`` left it, ``kv`` [rows, n_heads * (dim + vdim)] the expanded
+        keys of all heads, then the values; ``out`` [T, n_heads * vdim] bfloat16 (rows of single-
+        query tokens are left alone)."""
+        for t, nm in ((out, "out"), (q, "q"), (kv, "kv"), (rope, "rope")):
+            _want(t, nm, torch.bfloat16, 2)
+        _want(base, "base", torch.int32, 1)
+        T, rows = out.shape[0], kv.shape[0]
+        pad = -(-dim // 64) * 64
+        if out.shape[1] != n_heads * vdim or tuple(q.shape) != (T, n_heads * (pad + 64)) or \
+                kv.shape[1] != n_heads * (dim + vdim) or tuple(rope.shape) != (rows, 64):
+            raise KernelError("latent_prompt_attention: shapes do not fit")
+        self.launches += 1
+        _check(self.lib.hs_latent_prefill_tc(
+            _ptr(out), _ptr(q), _ptr(kv), _ptr(rope), _ptr(base), _ptr(plan.data),
+            4 + plan_decode_ints(plan.n_rows), plan.tile_cap, T, rows, n_heads, dim, rot_dim, vdim,
+            rank, int(window), float(scale), _ptr(status), self._stream()),
+            f"latent_prompt_attention(dim={dim},rot_dim={rot_dim},vdim={vdim})")
 
     # -- the gated delta rule ---------------------------------------------------------------
     @staticmethod

@@ -14,6 +14,10 @@ Rotary positions act on interleaved pairs of the rotated parts.  A layer built w
 ``shares_cache`` has no latent projection: it reads the rows another layer call wrote (the
 schedule names the entry) with its own queries, expansions and sink.
 
+Prompt portions inside a window may run in the other form (``latent_prompt_rows``): the latents of
+the positions they see are expanded to keys and values per head by one product, and the portion
+attends to those (dim + rot_dim and vdim numbers a query and key instead of 2 * kv_rank + rot_dim).
+
 With ``q_down`` the queries come through a latent of their own: ``c_q = rms_norm(W_dq h)`` of
 ``q_rank`` numbers, formed in the launch that writes the cache row (both latents are columns of
 one input projection), and the query matrix maps c_q instead of h.
@@ -90,6 +94,10 @@ class LatentAttention(Mixer):
         if wq.dtype == torch.bfloat16:
             self.w_absorb_nk = self.w_absorb.transpose(1, 2).contiguous()
             self.w_expand_nk = tensors[n["uv"]].view(self.H, self.V, self.R).contiguous()
+        # both expansions as one matrix, for the dense rows of windowed prompt portions
+        self.w_kv = None
+        if wq.dtype == torch.bfloat16 and self.window and not n["sink"]:
+            self.w_kv = torch.cat([tensors[n["uk"]], tensors[n["uv"]]]).contiguous()
         self.sink = tensors[n["sink"]] if n["sink"] else None
         self.w_out = tensors[n["o"]]
         i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
@@ -124,19 +132,54 @@ class LatentAttention(Mixer):
         if self.q_rank:
             q = ctx.buffer("latent_q", (T, self.q_width), torch.float32)
             ops.linear(q, cq, self.w_q_up)
+        att = ctx.buffer("latent_heads", (T, H * V), ctx.dtype)
+        only = {}
+        rows = self._prompt_rows(ctx)
+        if rows:
+            self._prompt_portions(ctx, att, q, cache, rows, rot)
+            if ctx.plan.decode_cap == 0:         # no single-query token in this step
+                ops.linear(x, att, self.w_out, None, residual=None if fresh else x)
+                return
+            only = {"singles": ctx.plan}
         qa = ctx.buffer("latent_qa", (T, H * R), torch.float32)
         ops.grouped_linear(qa, q, self.w_absorb, a_offset=0, a_group_stride=D + P,
-                           w_nk=self.w_absorb_nk)
+                           w_nk=self.w_absorb_nk, **only)
         lat = ctx.buffer("latent_mix", (T, H * R), torch.float32)
         if self.window:
             rot["window"] = self.window
+        if only:
+            rot["singles_only"] = True
         ops.latent_attention(lat, qa, q, cache.pool, cache.table, ctx.tok_pos, ctx.tok_req,
                              self.sink, n_heads=H, rank=R, rot_dim=P, qr_head_stride=D + P,
                              qr_offset=D, scale=self.scale, page_size=cache.page_size,
                              status=ctx.status, plan=ctx.plan, **rot)
-        att = ctx.buffer("latent_heads", (T, H * V), ctx.dtype)
-        ops.grouped_linear(att, lat, self.w_expand, w_nk=self.w_expand_nk)
+        ops.grouped_linear(att, lat, self.w_expand, w_nk=self.w_expand_nk, **only)
         ops.linear(x, att, self.w_out, None, residual=None if fresh else x)
+
+    def _prompt_rows(self, ctx) -> int:
+        """Dense rows the step's prompt portions need in expanded form; 0: not in that form."""
+        takes = getattr(ctx.ops, "latent_prompt_rows", None)
+        if self.w_kv is None or not self.q_rank or takes is None:
+            return 0
+        return takes(ctx.plan, ctx.n_requests, n_heads=self.H, dim=self.D, rot_dim=self.P,
+                     vdim=self.V, rank=self.R, window=self.window, scale=self.scale)
+
+    def _prompt_portions(self, ctx, att, q, cache, rows, rot):
+        ops, T = ctx.ops, q.shape[0]
+        H, D, P, V, R = self.H, self.D, self.P, self.V, self.R
+        lat = ctx.buffer("latent_dense", (rows, R), ctx.dtype)
+        rope = ctx.buffer("latent_dense_rot", (rows, 64), ctx.dtype)
+        qp = ctx.buffer("latent_q_padded", (T, H * (-(-D // 64) * 64 + 64)), ctx.dtype)
+        base = ctx.buffer("latent_base", (ctx.n_requests,), torch.int32)
+        ops.latent_gather(lat, rope, qp, base, q, cache.pool, cache.table, ctx.req_start,
+                          ctx.req_len, ctx.tok_pos, ctx.tok_req, n_heads=H, dim=D, rank=R,
+                          rot_dim=P, window=self.window, page_size=cache.page_size,
+                          status=ctx.status, **rot)
+        kv = ctx.buffer("latent_expanded", (rows, H * (D + V)), ctx.dtype)
+        ops.linear(kv, lat, self.w_kv)
+        ops.latent_prompt_attention(att, qp, kv, rope, base, ctx.plan, n_heads=H, dim=D, rot_dim=P,
+                                    vdim=V, rank=R, window=self.window, scale=self.scale,
+                                    status=ctx.status)
 
 
 register_mixer("latent_attention", LatentAttention)
