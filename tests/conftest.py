@@ -151,3 +151,20 @@ def mafuzen_case(request, mafuzen_cases):
 def mafuzen_planted(tmp_path_factory):
     import mafuzen_cases as mc
     return {which: mc.planted_case(tmp_path_factory, which) for which in mc.PLANTED}
+
+
+@pytest.fixture(scope="session")
+def pivinex_cases(tmp_path_factory):
+    import pivinex_cases as pc
+    return pc.make_cases(tmp_path_factory)
+
+
+@pytest.fixture(params=["case_a", "case_b"])
+def pivinex_case(request, pivinex_cases):
+    return pivinex_cases[request.param]
+
+
+@pytest.fixture(scope="session")
+def pivinex_planted(tmp_path_factory):
+    import pivinex_cases as pc
+    return {which: pc.planted_case(tmp_path_factory, which) for which in pc.PLANTED}
