@@ -5,8 +5,8 @@
 // `a` is float32 with row stride a_stride, so a group's input may be a slice of a wider row
 // (the unrotated part of one head's query, say); the weights are held k-major ([groups, k, n],
 // transposed once at binding) so that a warp's loads of one k are contiguous.  A block covers TT
-// tokens x 32 output columns; its four warps each sum a quarter of k for every column, and the
-// quarters are added in a fixed order, so a row's result depends on nothing else in the batch.
+// tokens x 32 output columns; its four or eight warps (the caller's choice) each sum their part of k for
+// every column, and the parts are added in a fixed order, so a row's result depends on nothing else in the batch.
 //
 // `list` (may be null): a step's attention plan; then row i of the launch is the i-th single-query
 // token of the plan (`n_tokens` bounds their number) and no other token is touched.
@@ -19,18 +19,18 @@ namespace hs {
 __device__ __forceinline__ int gl_token(const int* list, int i) { return list ? list[4 + 3 * i] : i; }
 
 constexpr int GL_TT = 8;          // tokens a block covers
-constexpr int GL_THREADS = 128;   // four warps: each takes a quarter of the summed index
 constexpr int GL_COLS = 32;       // output columns a block covers (one a lane)
 
-template <typename TW, typename TO>
-__global__ void __launch_bounds__(GL_THREADS)
+template <typename TW, typename TO, int GL_WARPS>
+__global__ void __launch_bounds__(32 * GL_WARPS)
 grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
                       const TW* __restrict__ w, int n_tokens, int a_stride, int a_off,
                       int a_gstride, int groups, int n, int k, const int* __restrict__ list) {
   extern __shared__ float s_a[];                    // [GL_TT][k]
   pdl_trigger();
   pdl_wait();
-  __shared__ float s_part[GL_THREADS / 32][GL_TT][GL_COLS];
+  __shared__ float s_part[GL_WARPS][GL_TT][GL_COLS];
+  constexpr int GL_THREADS = 32 * GL_WARPS;
   const int t0 = blockIdx.x * GL_TT;
   if (list) n_tokens = min(n_tokens, list[0]);
   if (t0 >= n_tokens) return;
@@ -48,11 +48,11 @@ grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
   float acc[GL_TT];
 #pragma unroll
   for (int tt = 0; tt < GL_TT; ++tt) acc[tt] = 0.f;
-  const int per = (k + 3) / 4;
+  const int per = (k + GL_WARPS - 1) / GL_WARPS;
   const int k_lo = warp * per, k_hi = min(k, k_lo + per);
   if (j < n) {
     const TW* wg = w + (size_t)g * k * n + j;
-#pragma unroll 8
+#pragma unroll 16
     for (int kk = k_lo; kk < k_hi; ++kk) {
       const float wv = to_f(wg[(size_t)kk * n]);
 #pragma unroll
@@ -62,12 +62,14 @@ grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
 #pragma unroll
   for (int tt = 0; tt < GL_TT; ++tt) s_part[warp][tt][lane] = acc[tt];
   __syncthreads();
-  // the four quarters are added in a fixed order: a row's sum never depends on the batch
+  // the shares of the warps are added in a fixed order: a row's sum never depends on the batch
   for (int i = threadIdx.x; i < GL_TT * GL_COLS; i += GL_THREADS) {
     const int tt = i / GL_COLS, c = i - tt * GL_COLS;
     const int col = blockIdx.z * GL_COLS + c;
     if (tt < nt && col < n) {
-      const float v = ((s_part[0][tt][c] + s_part[1][tt][c]) + s_part[2][tt][c]) + s_part[3][tt][c];
+      float v = s_part[0][tt][c];
+#pragma unroll
+      for (int q = 1; q < GL_WARPS; ++q) v += s_part[q][tt][c];
       out[(size_t)gl_token(list, t0 + tt) * groups * n + (size_t)g * n + col] = from_f<TO>(v);
     }
   }
@@ -213,8 +215,9 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
 
 HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_tokens,
                                 int a_stride, int a_off, int a_gstride, int groups, int n, int k,
-                                int w_dtype, int out_dtype, const int* list, void* stream) {
-  if (!out || !a || !w) return HS_ERR_ARGUMENT;
+                                int w_dtype, int out_dtype, const int* list, int parts,
+                                void* stream) {
+  if (!out || !a || !w || (parts != 4 && parts != 8)) return HS_ERR_ARGUMENT;
   if (groups <= 0 || n <= 0 || k <= 0) return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
   const size_t smem = (size_t)hs::GL_TT * k * sizeof(float);
@@ -222,18 +225,24 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
   dim3 grid((n_tokens + hs::GL_TT - 1) / hs::GL_TT, groups, (n + hs::GL_COLS - 1) / hs::GL_COLS);
   cudaStream_t st = (cudaStream_t)stream;
   cudaError_t e = cudaSuccess;
-#define HS_GL(TW, TO)                                                                         \
+#define HS_GL_AS(TW, TO, NW)                                                                  \
   do {                                                                                        \
-    auto kern = hs::grouped_linear_kernel<TW, TO>;                                            \
+    auto kern = hs::grouped_linear_kernel<TW, TO, NW>;                                        \
     if (smem > 48 * 1024)                                                                     \
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
-    e = hs_launch(kern, grid, dim3(hs::GL_THREADS), smem, st, hs_pdl_enabled(), (TO*)out, a, \
+    e = hs_launch(kern, grid, dim3(32 * NW), smem, st, hs_pdl_enabled(), (TO*)out, a,         \
                   (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, list);    \
+  } while (0)
+#define HS_GL(TW, TO)                                                                         \
+  do {                                                                                        \
+    if (parts == 8) HS_GL_AS(TW, TO, 8);                                                      \
+    else HS_GL_AS(TW, TO, 4);                                                                 \
   } while (0)
   if (w_dtype == HS_DT_F32 && out_dtype == HS_DT_F32) HS_GL(float, float);
   else if (w_dtype == HS_DT_BF16 && out_dtype == HS_DT_F32) HS_GL(__nv_bfloat16, float);
   else if (w_dtype == HS_DT_BF16 && out_dtype == HS_DT_BF16) HS_GL(__nv_bfloat16, __nv_bfloat16);
   else return HS_ERR_UNSUPPORTED;
+#undef HS_GL_AS
 #undef HS_GL
   return e == cudaSuccess ? HS_OK : (int)e;
 }

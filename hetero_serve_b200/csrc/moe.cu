@@ -206,7 +206,7 @@ moe_route_top_kernel(int* __restrict__ sel_idx, float* __restrict__ sel_w,
 // token forms the logits first and its warp 0 chooses.  The logits lie in shared memory, the
 // statistics of the softmax are formed in an order fixed by E.
 template <typename TH>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 moe_route_softmax_kernel(int* __restrict__ sel_idx, float* __restrict__ sel_w,
                          const TH* __restrict__ h, const float* __restrict__ w_router,
                          const float* __restrict__ correction, const int* __restrict__ tok_req,
@@ -697,8 +697,7 @@ HS_EXPORT int hs_moe_route_softmax(int* sel_idx, float* sel_w, const void* h,
   if (!sel_idx || !sel_w || !h || !w_router || !tok_req) return HS_ERR_ARGUMENT;
   if (width <= 0 || E <= 0 || top <= 0 || top > E) return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
-  int warps = (E + 3) / 4;                       // four experts a warp, up to eight warps
-  warps = z_in ? 4 : (warps < 1 ? 1 : (warps > 8 ? 8 : warps));
+  const int warps = z_in ? 4 : (E > 32 ? 32 : E);           // a warp an output, up to 32
   const size_t smem = (z_in ? (size_t)warps * 2 * E : (size_t)2 * E + width) * sizeof(float);
   if (smem > 48 * 1024) return HS_ERR_UNSUPPORTED;
   const dim3 grid(z_in ? (n_tokens + warps - 1) / warps : n_tokens);

@@ -200,8 +200,9 @@ def _declare(lib) -> None:
         "hs_dyt_norm": [P, P, P, P, P, I, I, F, I, P],
         "hs_scale": [P, ctypes.c_longlong, F, P],
         "hs_rotary_pairs": [P, P, P, P, I, I, I, I, I, I, P],
-        "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P, P],
+        "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P, I, P],
         "hs_grouped_linear_mma": [P, P, P, I, I, I, I, I, I, I, I, I, P, P],
+        "hs_latent_decode_mma": [P] * 7 + [I] * 7 + [F, I, I, I, P, P, I, I, P],
         "hs_latent_prefill_tc_takes": [I, I, I, I, I, F],
         "hs_latent_gather": [P] * 11 + [I] * 12 + [P, I, P, P],
         "hs_latent_prefill_tc": [P] * 6 + [I] * 10 + [F, P, P],
@@ -344,6 +345,7 @@ class CudaOps:
         self._moe_need: dict = {}
         # windowed latent attention of prompt portions in expanded form, on tcgen05 tensor cores
         self.latent_expanded = True
+        self.latent_decode_mma = True   # single-query tokens of latent attention likewise
         self.latent_mma = True      # prompt portions of latent attention on the tensor cores
         self.biased_mma = True      # prompt portions of the biased chunk attention likewise
         self.pooled_mma = True      # ... and of the attention over a window and pooled blocks
@@ -1066,7 +1068,7 @@ class CudaOps:
                "rotary_pairs")
 
     def grouped_linear(self, out, a, w, *, a_offset=0, a_group_stride=None, w_nk=None,
-                       exact=False, singles=None):
+                       exact=False, singles=None, parts=4):
         """Block-diagonal linear: ``out[t, g*n + j] = sum_k a[t, a_offset + g*a_group_stride + k]
         * w[g, k, j]``.  ``a`` float32 (a group's input may be a slice of a wider row), ``w``
         [groups, k, n] (k-major), ``out`` [T, groups * n] float32 or of w's type.  ``w_nk`` is
@@ -1075,7 +1077,8 @@ class CudaOps:
         ``exact`` ``a`` enters as the sum of three bfloat16 terms, which loses nothing of a
         float32: for weights that are bfloat16 numbers the result is then the float32 product,
         and ``out`` is float32).  With ``singles`` (the step's attention plan) only the plan's
-        single-query tokens are worked on."""
+        single-query tokens are worked on.  ``parts`` (4 or 8): in how many pieces the CUDA-core
+        kernel cuts the summed index of a few tokens' rows (the order of its additions)."""
         _want(a, "a", torch.float32, 2)
         _want(w, "w", _FLOATS, 3)
         _want(out, "out", _FLOATS, 2)
@@ -1105,7 +1108,7 @@ class CudaOps:
                 return
         _check(self.lib.hs_grouped_linear(_ptr(out), _ptr(a), _ptr(w), T, a.shape[1],
                                           int(a_offset), gs, groups, n, k, _DT[w.dtype],
-                                          _DT[out.dtype], _ptr(listed), self._stream()),
+                                          _DT[out.dtype], _ptr(listed), int(parts), self._stream()),
                f"grouped_linear(groups={groups},n={n},k={k})")
 
     # -- attention over a shared latent ---------------------------------------------------
@@ -1158,8 +1161,10 @@ class CudaOps:
         ``qr[t, qr_offset + h * qr_head_stride : + rot_dim]``; with ``freq`` it arrives
         unrotated and its first ``rot_dims`` entries are rotated as they are read.  With the
         step's ``plan`` and a bfloat16 cache, the plan's tiles (prompt portions) run on the
-        tensor cores with the queries rounded to bfloat16, its single-query tokens on the CUDA
-        cores; without a plan every token runs on the CUDA cores.  With ``singles_only`` the
+        tensor cores with the queries rounded to bfloat16, its single-query tokens on the tensor
+        cores with queries and weights in several bfloat16 terms (float32's mantissa), a cluster of
+        blocks a token; without a plan, in float32 and for sizes those kernels do not take, tokens
+        run on the CUDA cores.  With ``singles_only`` the
         plan's tiles are left out (another operation serves them)."""
         _want(out, "out", torch.float32, 2)
         _want(qa, "qa", torch.float32, 2)
@@ -1200,6 +1205,18 @@ class CudaOps:
                     return
                 listed = plan.data          # the CUDA-core kernel takes the single-query tokens
                 n = plan.decode_cap
+        if (plan is not None and pool.dtype == torch.bfloat16 and self.tensor_cores
+                and self.latent_decode_mma and (listed is not None or plan.tile_cap == 0)
+                and plan.decode_cap > 0):
+            code = self.lib.hs_latent_decode_mma(
+                _ptr(out), _ptr(qa), _ptr(qr), _ptr(pool), _ptr(table), _ptr(sink),
+                _ptr(plan.data), plan.decode_cap, n_heads, rank, rot_dim, qr.shape[1],
+                int(qr_head_stride), int(qr_offset), float(scale), page_size, n_pages,
+                table.shape[1], _ptr(status), _ptr(freq), rot, int(window), self._stream())
+            if code != -1:
+                _check(code, f"latent_decode_mma(rank={rank},rot_dim={rot_dim})")
+                self.launches += 1
+                return
         # few tokens: the keys of each are split over several blocks so that the device fills
         blocks = n * -(-n_heads // 8)
         nsplit = 1 if blocks >= self.sm_count else min(16, -(-2 * self.sm_count // blocks))

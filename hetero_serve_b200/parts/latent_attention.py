@@ -143,7 +143,7 @@ class LatentAttention(Mixer):
             only = {"singles": ctx.plan}
         qa = ctx.buffer("latent_qa", (T, H * R), torch.float32)
         ops.grouped_linear(qa, q, self.w_absorb, a_offset=0, a_group_stride=D + P,
-                           w_nk=self.w_absorb_nk, **only)
+                           w_nk=self.w_absorb_nk, parts=8, **only)
         lat = ctx.buffer("latent_mix", (T, H * R), torch.float32)
         if self.window:
             rot["window"] = self.window
@@ -153,7 +153,7 @@ class LatentAttention(Mixer):
                              self.sink, n_heads=H, rank=R, rot_dim=P, qr_head_stride=D + P,
                              qr_offset=D, scale=self.scale, page_size=cache.page_size,
                              status=ctx.status, plan=ctx.plan, **rot)
-        ops.grouped_linear(att, lat, self.w_expand, w_nk=self.w_expand_nk, **only)
+        ops.grouped_linear(att, lat, self.w_expand, w_nk=self.w_expand_nk, parts=8, **only)
         ops.linear(x, att, self.w_out, None, residual=None if fresh else x)
 
     def _prompt_rows(self, ctx) -> int:

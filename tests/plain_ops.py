@@ -163,7 +163,7 @@ class PlainOps:
                 buf[t, lo:lo + dims] = seg.to(buf.dtype)
 
     def grouped_linear(self, out, a, w, *, a_offset=0, a_group_stride=None, w_nk=None, exact=False,
-                       singles=None):
+                       singles=None, parts=4):
         groups, k, n = w.shape
         gs = k if a_group_stride is None else a_group_stride
         T = out.shape[0]

@@ -104,15 +104,16 @@ def test_windowed_latent_attention_on_the_cuda_cores(ops, plain, window, dtype, 
                                               (512, 64, 16), (24, 8, 1), (40, 2, 17)])
 @pytest.mark.parametrize("window", [1, 17, 64, 300])
 def test_windowed_latent_attention_of_single_tokens_by_list(ops, plain, rank, rot, heads, window):
-    """A step of single tokens with a plan and a bfloat16 cache."""
+    """A step of single tokens with a plan and a bfloat16 cache: queries and weights keep float32's
+    mantissa on the tensor cores too."""
     b = Batch([(0, 1), (5, 1), (63, 2), (64, 1), (299, 1), (300, 1), (350, 4), (16, 3)], rank + rot, window,
               BF16, seed=40 + window)
     plan = ops.make_plan(b.host, b.n, PAGE)
     assert plan.tile_cap == 0 and plan.decode_cap == b.n
     got, want = attend(ops, plain, b, heads, rank, rot, scale=0.2, plan=plan)
-    close(got, want, 2e-2)
+    close(got, want, 2e-5)
     got, want = attend(ops, plain, b, heads, rank, rot, scale=0.2, plan=plan, sink=rnd(heads, seed=3))
-    close(got, want, 2e-2)
+    close(got, want, 2e-5)
 
 
 @pytest.mark.parametrize("rank, rot, heads", [(32, 8, 3), (272, 24, 5), (16, 4, 70)])
