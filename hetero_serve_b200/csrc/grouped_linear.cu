@@ -228,7 +228,7 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
 #define HS_GL_AS(TW, TO, NW)                                                                  \
   do {                                                                                        \
     auto kern = hs::grouped_linear_kernel<TW, TO, NW>;                                        \
-    if (smem > 48 * 1024)                                                                     \
+    if (smem > 32 * 1024)  /* with the static array a block may then pass 48 KB */            \
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     e = hs_launch(kern, grid, dim3(32 * NW), smem, st, hs_pdl_enabled(), (TO*)out, a,         \
                   (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, list);    \

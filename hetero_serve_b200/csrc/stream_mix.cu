@@ -240,7 +240,7 @@ HS_EXPORT int hs_embed_norm(float* x, float* x0, const int* ids, const int* req,
   const void* ptrs[] = {x, x0, table, g, b, out, g2, b2};
   const bool vec = hs::sm_vec(width, ptrs, 8);
   const size_t smem = vec ? 0 : (size_t)width * sizeof(float);
-  if (smem > 48 * 1024) return HS_ERR_UNSUPPORTED;
+  if (smem > 47 * 1024) return HS_ERR_UNSUPPORTED;
   const dim3 grid(n_tokens), block(hs::sm_threads(width, vec));
   cudaStream_t st = (cudaStream_t)stream;
 #define HS_EN(VEC, T, TO)                                                                        \
@@ -274,7 +274,7 @@ HS_EXPORT int hs_residual_mix(float* x, const float* y1, const float* s1, const 
   const void* ptrs[] = {x, y1, s1, y2, s2, again, out, g, b};
   const bool vec = hs::sm_vec(width, ptrs, 9);
   const size_t smem = vec ? 0 : (size_t)width * sizeof(float);
-  if (smem > 48 * 1024) return HS_ERR_UNSUPPORTED;
+  if (smem > 47 * 1024) return HS_ERR_UNSUPPORTED;
   const dim3 grid(n_rows), block(hs::sm_threads(width, vec));
   cudaStream_t st = (cudaStream_t)stream;
   cudaError_t e = cudaSuccess;

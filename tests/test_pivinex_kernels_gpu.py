@@ -101,7 +101,8 @@ def test_windowed_latent_attention_on_the_cuda_cores(ops, plain, window, dtype, 
 
 
 @pytest.mark.parametrize("rank, rot, heads", [(32, 8, 3), (64, 16, 8), (272, 24, 5), (16, 4, 20),
-                                              (512, 64, 16), (24, 8, 1), (40, 2, 17)])
+                                              (512, 64, 16), (24, 8, 1), (40, 2, 17),
+                                              (128, 64, 2), (120, 80, 3)])
 @pytest.mark.parametrize("window", [1, 17, 64, 300])
 def test_windowed_latent_attention_of_single_tokens_by_list(ops, plain, rank, rot, heads, window):
     """A step of single tokens with a plan and a bfloat16 cache: queries and weights keep float32's
