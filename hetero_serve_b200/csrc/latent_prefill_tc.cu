@@ -98,26 +98,32 @@ latent_gather_kernel(__nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict_
   const int r = tok_req[t];
   if (r < 0 || req_len[r] <= max_single) return;
   const int pos = tok_pos[t];
+  __shared__ float2 s_cs[32];                            // cosine and sine of a turned pair
+  if ((int)threadIdx.x < rot_dims / 2)
+    pair_angle(pos, freq[threadIdx.x], &s_cs[threadIdx.x].x, &s_cs[threadIdx.x].y);
+  __syncthreads();
   const int qw = q_pad_d + 64;                           // padded numbers a head
   const float* src = q + (size_t)t * q_stride;
   __nv_bfloat16* dst = q_out + (size_t)t * n_heads * qw;
   for (int i = threadIdx.x; i < n_heads * qw / 2; i += THREADS) {
     const int h = 2 * i / qw, e = 2 * i - h * qw;        // a pair of neighbours
     const float* s = src + (size_t)h * (D + P);
-    float v[2];
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      const int c = e + x;
-      v[x] = 0.f;
-      if (c < D) {
-        v[x] = s[c];
-      } else if (c >= q_pad_d && c - q_pad_d < P) {
-        const int k = c - q_pad_d;
-        v[x] = k < rot_dims ? rotate_entry(s[D + k], s[D + (k ^ 1)], k, rot_dims, pos, freq)
-                            : s[D + k];
+    float x = 0.f, y = 0.f;
+    if (e < D) {                                         // D is even
+      x = s[e];
+      y = s[e + 1];
+    } else if (e >= q_pad_d && e - q_pad_d < P) {
+      const int k = e - q_pad_d;
+      x = s[D + k];
+      y = k + 1 < P ? s[D + k + 1] : 0.f;
+      if (k < rot_dims) {
+        const float2 cs = s_cs[k >> 1];
+        const float a = x * cs.x - y * cs.y;
+        y = y * cs.x + x * cs.y;
+        x = a;
       }
     }
-    *(__nv_bfloat162*)(dst + 2 * i) = __floats2bfloat162_rn(v[0], v[1]);
+    *(__nv_bfloat162*)(dst + 2 * i) = __floats2bfloat162_rn(x, y);
   }
 }
 
@@ -460,7 +466,7 @@ HS_EXPORT int hs_latent_gather(void* lat, void* rope, void* q_out, int* base, co
       !tok_pos || !tok_req || !status)
     return HS_ERR_ARGUMENT;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > P || (rot_dims && !freq)) return HS_ERR_ARGUMENT;
-  if (window <= 0 || R <= 0 || P <= 0 || P > 64 || D <= 0 || n_heads <= 0 || page_size <= 0)
+  if (window <= 0 || R <= 0 || P <= 0 || P > 64 || D <= 0 || D % 2 || n_heads <= 0 || page_size <= 0)
     return HS_ERR_UNSUPPORTED;
   if (n_requests <= 0 || n_tokens <= 0) return HS_OK;
   const int pad = (D + 63) / 64 * 64;

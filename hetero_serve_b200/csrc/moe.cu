@@ -49,6 +49,7 @@ __device__ __forceinline__ float row_dot(const float* __restrict__ w, const floa
                                          int lane) {
   float acc = 0.f;
   if ((n & 3) == 0 && (((uintptr_t)w) & 15) == 0) {
+#pragma unroll 8
     for (int k = lane * 4; k < n; k += 128) {
       const float4 a = *(const float4*)(w + k);
       acc = fmaf(a.x, v[k], acc); acc = fmaf(a.y, v[k + 1], acc);
@@ -624,6 +625,49 @@ __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restric
   pdl_wait();
   const int t = blockIdx.x;
   if (tok_req[t] < 0) return;
+  if (width % 4 == 0 && top <= MAX_TOP_AT_ONCE && !((uintptr_t)x & 15) && !((uintptr_t)h & 7)) {
+    // four columns a thread, the rows of all choices on their way before the first sum
+    int at[MAX_TOP_AT_ONCE];
+    float w[MAX_TOP_AT_ONCE];
+#pragma unroll
+    for (int k = 0; k < MAX_TOP_AT_ONCE; ++k) {
+      at[k] = -1;
+      w[k] = 0.f;
+      if (k < top) {
+        at[k] = pair_pos[(size_t)t * top + k];
+        w[k] = sel_w[(size_t)t * top + k];
+        const int e = n_identity ? sel_idx[(size_t)t * top + k] : -1;
+        if (at[k] < 0 && e >= E && e < E + n_identity) at[k] = -2;      // the input itself
+      }
+    }
+    for (int n = 4 * threadIdx.x; n < width; n += 4 * blockDim.x) {
+      float4 v[MAX_TOP_AT_ONCE];
+#pragma unroll
+      for (int k = 0; k < MAX_TOP_AT_ONCE; ++k) {
+        if (at[k] >= 0) {
+          v[k] = *(const float4*)(rows + (size_t)at[k] * width + n);
+        } else if (at[k] == -2) {
+          const __nv_bfloat162* p = (const __nv_bfloat162*)(h + (size_t)t * width + n);
+          const float2 a = __bfloat1622float2(p[0]), b = __bfloat1622float2(p[1]);
+          v[k] = make_float4(a.x, a.y, b.x, b.y);
+        }
+      }
+      float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < MAX_TOP_AT_ONCE; ++k)
+        if (at[k] != -1) {
+          sum.x = fmaf(w[k], v[k].x, sum.x); sum.y = fmaf(w[k], v[k].y, sum.y);
+          sum.z = fmaf(w[k], v[k].z, sum.z); sum.w = fmaf(w[k], v[k].w, sum.w);
+        }
+      float4* dst = (float4*)(x + (size_t)t * width + n);
+      if (accumulate) {
+        const float4 o = *dst;
+        sum.x += o.x; sum.y += o.y; sum.z += o.z; sum.w += o.w;
+      }
+      *dst = sum;
+    }
+    return;
+  }
   for (int n = threadIdx.x; n < width; n += blockDim.x) {
     float sum = 0.f;
     for (int k = 0; k < top; ++k) {
