@@ -5,3 +5,4 @@ from . import putelix  # noqa: F401
 from . import roritar  # noqa: F401
 from . import mafuzen  # noqa: F401
 from . import pivinex  # noqa: F401
+from . import nukodra  # noqa: F401

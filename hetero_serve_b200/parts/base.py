@@ -3,7 +3,7 @@
 A part is built from the parameters of its :class:`PartSpec` alone.  It says which
 checkpoint tensors it needs (:meth:`Part.tensor_requests`), receives them converted
 and on the device (:meth:`Part.bind`) and runs on a :class:`StepContext`
-(``hetero_serve_b200.engine.context``).  Six kinds exist:
+(``hetero_serve_b200.engine.context``).  These kinds exist:
 
 ========  ==================================================================
 mixer     ``forward(ctx, h, x, cache)``: mixes information between the tokens
@@ -13,6 +13,8 @@ feed      ``forward(ctx, h, x)``: per-token transform, added into ``x``.
 norm      ``forward(ctx, out, x, rows=None)``: normalises rows of ``x``.
 scale     ``factor``: a float32 vector [width] an arrangement multiplies a
           sublayer's output with, column by column, before it is added.
+connection  learned tables with which an arrangement lets a sublayer read and write
+          several copies of the stream.
 position  how positions enter: a table added at the embedding and/or a
           transform of queries and keys inside a mixer.
 embedding / head: token table at the input, logits at the output.
@@ -163,8 +165,8 @@ class Head(Part):
 
 
 _REGISTRIES: dict[str, dict[str, Callable[..., Part]]] = {
-    "mixer": {}, "feed_forward": {}, "norm": {}, "scale": {}, "position": {}, "embedding": {},
-    "head": {},
+    "mixer": {}, "feed_forward": {}, "norm": {}, "scale": {}, "connection": {}, "position": {},
+    "embedding": {}, "head": {},
 }
 
 
@@ -189,6 +191,10 @@ def register_norm(kind, factory, *, replace=False):
 
 def register_scale(kind, factory, *, replace=False):
     _register("scale", kind, factory, replace)
+
+
+def register_connection(kind, factory, *, replace=False):
+    _register("connection", kind, factory, replace)
 
 
 def register_position(kind, factory, *, replace=False):

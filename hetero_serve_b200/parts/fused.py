@@ -75,7 +75,7 @@ def plan_fused_decode(model, ops, storage, page_size: int):
     layers, sizes = [], None
     for call in model.schedule:
         block = model.blocks[call.layer]
-        if type(block) is not PreNormBlock or not call.writes_cache:
+        if type(block) is not PreNormBlock or not call.writes_cache or block.feed_forward is None:
             return None
         n1, mx = block.norm1.fused_decode_params(), block.mixer.fused_decode_params()
         n2, ff = block.norm2.fused_decode_params(), block.feed_forward.fused_decode_params()

@@ -54,9 +54,16 @@ class Block:
 
 class PreNormBlock(Block):
     """x += mixer(norm1(x)); x += feed_forward(norm2(x))
-    (heteroserve/model/torch_engine.py:297-317)."""
+    (heteroserve/model/torch_engine.py:297-317).  A layer may leave ``norm2`` and
+    ``feed_forward`` out (both or neither): it then ends after the mixer."""
 
     slots = {"norm1": "norm", "mixer": "mixer", "norm2": "norm", "feed_forward": "feed_forward"}
+    optional = ("norm2", "feed_forward")
+
+    def __init__(self, spec: LayerSpec):
+        super().__init__(spec)
+        if (self.norm2 is None) != (self.feed_forward is None):
+            raise ValueError("arrangement 'pre_norm': norm2 and feed_forward come together")
 
     def forward(self, ctx, x, cache):
         h = ctx.buffer("normed", (x.shape[0], x.shape[1]), ctx.dtype)
@@ -65,6 +72,8 @@ class PreNormBlock(Block):
         else:
             self.norm1.forward(ctx, h, x)
             self.mixer.forward(ctx, h, x, cache)
+        if self.feed_forward is None:
+            return
         if self.feed_forward.takes_norm:
             self.feed_forward.forward(ctx, h, x, norm=self.norm2)
         else:
@@ -252,11 +261,95 @@ class ScaledParallelBlock(Block):
         ctx.embedding_added = ctx.next_adds_embedding
 
 
+class HyperConnectedBlock(Block):
+    """Two sublayers behind norms that read and write several copies of the stream:
+
+        u = read1 . X;  X <- mix1(X) + write1 * mixer(norm1(u))
+        u = read2 . X;  X <- mix2(X) + write2 * feed_forward(norm2(u))
+
+    with the tables of one ``connection`` part per sublayer (``hyper_connection``).  The copies of
+    a token are neighbours in one float32 row; they live in the step context from block to block
+    of this arrangement.  In front of the first such block every copy equals the stream, behind
+    the last one the stream is the sum of the copies, so blocks of other arrangements may stand
+    anywhere between.  One launch behind each sublayer updates all copies and forms the norm of
+    what the next sublayer reads.  A layer may leave ``norm2``, ``feed_forward`` and ``connect2``
+    out (all or none)."""
+
+    slots = {"norm1": "norm", "mixer": "mixer", "connect1": "connection", "norm2": "norm",
+             "feed_forward": "feed_forward", "connect2": "connection"}
+    optional = ("norm2", "feed_forward", "connect2")
+
+    def __init__(self, spec: LayerSpec):
+        super().__init__(spec)
+        present = [getattr(self, n) is not None for n in self.optional]
+        if any(present) != all(present):
+            raise ValueError("arrangement 'hyper_connected': norm2, feed_forward and connect2 "
+                             "come together")
+        self.streams = self.connect1.streams
+        if self.connect2 is not None and self.connect2.streams != self.streams:
+            raise ValueError("arrangement 'hyper_connected': both sublayers connect to the same "
+                             "number of streams")
+
+    @staticmethod
+    def _reads(ctx, norm, h, u, connection, more):
+        """Completes the arguments of a launch that also forms norm(read . X) into h; returns
+        whether the norm is left to its own launch."""
+        row = getattr(norm, "rms_row", None)
+        more["read"] = connection.read
+        if row is not None:
+            more.update(out=h, norm=row())
+            return False
+        more["u"] = u
+        return True
+
+    def forward(self, ctx, x, cache):
+        T, W = x.shape
+        X = ctx.buffer("streams", (T, self.streams * W), torch.float32)
+        h = ctx.buffer("normed", (T, W), ctx.dtype)
+        u = ctx.buffer("connected", (T, W), torch.float32)
+        y = ctx.buffer("sublayer_out", (T, W), torch.float32)
+        # in front of the first such block the copies are equal: the stream stands for all
+        source = X if ctx.live_streams == self.streams else x
+        if source is x or not ctx.normed_ahead:
+            more = {}
+            alone = self._reads(ctx, self.norm1, h, u, self.connect1, more)
+            ctx.ops.hyper_mix(None, source, streams=self.streams, **more)
+            if alone:
+                self.norm1.forward(ctx, h, u)
+        out = OutputNormBlock._run(self.mixer, ctx, h, y, cache)
+        if self.feed_forward is not None:
+            more = {}
+            alone = self._reads(ctx, self.norm2, h, u, self.connect2, more)
+            ctx.ops.hyper_mix(X, source, out, streams=self.streams, mix=self.connect1.mix,
+                              write=self.connect1.write, **more)
+            if alone:
+                self.norm2.forward(ctx, h, u)
+            source = X
+            out = OutputNormBlock._run(self.feed_forward, ctx, h, y)
+            last = self.connect2
+        else:
+            last = self.connect1
+        nxt, more = ctx.next_block, {}
+        follows = isinstance(nxt, HyperConnectedBlock) and nxt.streams == self.streams \
+            and not ctx.next_adds_embedding
+        if follows:
+            ctx.normed_ahead = not self._reads(ctx, nxt.norm1, h, u, nxt.connect1, more)
+            if not ctx.normed_ahead:
+                more = {}
+        else:
+            more["u"] = x                         # the sum of the copies
+            ctx.normed_ahead = False
+        ctx.ops.hyper_mix(X if follows else None, source, out, streams=self.streams,
+                          mix=last.mix, write=last.write, **more)
+        ctx.live_streams = self.streams if follows else 0
+
+
 _ARRANGEMENTS: dict[str, Callable[[LayerSpec], Block]] = {"pre_norm": PreNormBlock,
                                                           "parallel": ParallelBlock,
                                                           "output_norm": OutputNormBlock,
                                                           "sandwich_norm": SandwichNormBlock,
-                                                          "scaled_parallel": ScaledParallelBlock}
+                                                          "scaled_parallel": ScaledParallelBlock,
+                                                          "hyper_connected": HyperConnectedBlock}
 
 
 def register_arrangement(name: str, factory: Callable[[LayerSpec], Block], *, replace=False):
@@ -407,6 +500,7 @@ class Model:
         ctx.position = self.position          # mixers ask it whether it acts on queries and keys
         ctx.stream_copy_fresh = False         # no copy of the stream in the compute type yet
         ctx.normed_ahead = False              # nobody has formed the next block's first norm
+        ctx.live_streams = 0                  # copies of the stream that live beside it
         ctx.embedding_added = False           # nobody has added what a call wants added before it
         ctx.embedding_output = None
         first = self.schedule[0] if self.schedule else None

@@ -43,6 +43,11 @@ class RMSNorm(Norm):
         # the fused add takes plain weights: one-plus weights are formed once
         self.add_weight = (1.0 + self.weight) if self.one_plus else self.weight
 
+    def rms_row(self):
+        """(weight, eps) with plain weights, for a launch that forms this norm of rows it has at
+        hand."""
+        return self.add_weight, self.eps
+
     def forward(self, ctx, out, x, rows=None):
         ctx.ops.rms_norm(out, x, self.weight, self.eps, rows, one_plus=self.one_plus)
 

@@ -163,13 +163,16 @@ class PlainOps:
                 buf[t, lo:lo + dims] = seg.to(buf.dtype)
 
     def grouped_linear(self, out, a, w, *, a_offset=0, a_group_stride=None, w_nk=None, exact=False,
-                       singles=None, parts=4):
+                       singles=None, parts=4, gate=None, gate_offset=0):
         groups, k, n = w.shape
         gs = k if a_group_stride is None else a_group_stride
         T = out.shape[0]
         for g in range(groups):
             lo = a_offset + g * gs
             v = a[:T, lo:lo + k].to(self.cd) @ w[g].to(self.cd)
+            if gate is not None:
+                lo = gate_offset + g * n
+                v = v * torch.sigmoid(gate[:T, lo:lo + n].to(self.cd))
             out[:, g * n:(g + 1) * n] = v.to(out.dtype)
 
     def _turned(self, vec, position, freq, rot_dims):
@@ -713,40 +716,49 @@ class PlainOps:
             sel_w[t] = 1.0 / top
 
     def head_norm_gate(self, out, o, weight, gate, *, gate_offset, heads, dim, eps,
-                       gate_act="silu", out_scale=1.0):
+                       gate_act="silu", out_scale=1.0, gate_first=False):
         n = out.shape[0]
-        v = self._rms(o[:n].to(self.cd).view(n, heads, dim), eps).reshape(n, heads * dim)
+        v = o[:n].to(self.cd)
+        if gate is not None and gate_first:
+            v = v * _GATE[gate_act](gate[:n, gate_offset:gate_offset + heads * dim].to(self.cd))
+        v = self._rms(v.reshape(n, heads, dim), eps).reshape(n, heads * dim)
         if weight is not None:
             v = v * weight.to(self.cd)
-        if gate is not None:
+        if gate is not None and not gate_first:
             v = v * _GATE[gate_act](gate[:n, gate_offset:gate_offset + heads * dim].to(self.cd))
         out.copy_((v * out_scale).to(out.dtype))
 
     def span_prepare(self, q_out, pool, proj, table, tok_pos, tok_req, *, n_heads, n_kv_heads,
                      head_dim, value_dim, q_off, k_off, v_off, qk_norm, eps, writes, page_size,
-                     status):
+                     status, wq=None, wk=None, freq=None, rot_dims=0):
         H, G, D, V = n_heads, n_kv_heads, head_dim, value_dim
         pv = pool.view(-1, G, page_size, D + V)
+
+        def formed(x, w, heads, pos):
+            if w is not None:
+                x = self._rms(x, eps) * w.to(self.cd)      # over the whole projection
+            x = x.view(heads, D)
+            return self._turn_halves(self._rms(x, eps) if qk_norm else x, pos, freq, rot_dims)
+
         for t in range(q_out.shape[0]):
             r = int(tok_req[t])
             if r < 0:
                 continue
             row = proj[t].to(self.cd)
-            q = row[q_off:q_off + H * D].view(H, D)
-            q_out[t] = (self._rms(q, eps) if qk_norm else q).reshape(-1).to(q_out.dtype)
+            p = int(tok_pos[t])
+            q_out[t] = formed(row[q_off:q_off + H * D], wq, H, p).reshape(-1).to(q_out.dtype)
             if not writes:
                 continue
-            k = row[k_off:k_off + G * D].view(G, D)
-            v = k if v_off is None else row[v_off:v_off + G * V].view(G, V)
-            kn = self._rms(k, eps) if qk_norm else k
-            p = int(tok_pos[t])
+            k = row[k_off:k_off + G * D]
+            v = k.view(G, D) if v_off is None else row[v_off:v_off + G * V].view(G, V)
+            kn = formed(k, wk, G, p)
             page = int(table[r, p // page_size])
             pv[page, :, p % page_size, :D] = kn.to(pool.dtype)
             pv[page, :, p % page_size, D:] = v.to(pool.dtype)
 
     def span_attention(self, out, q, pool, table, tok_pos, tok_req, *, n_heads, n_kv_heads,
                        head_dim, value_dim, scale, slopes, window, keep_first, gate, gate_offset,
-                       out_scale, page_size, status, plan=None):
+                       out_scale, page_size, status, plan=None, softcap=0.0, sinks=None):
         H, G, D, V = n_heads, n_kv_heads, head_dim, value_dim
         pv = pool.view(-1, G, page_size, D + V)
         for t in range(out.shape[0]):
@@ -765,11 +777,108 @@ class PlainOps:
                 s = (rows[:, g, :D] @ qt[hd]) * scale
                 if slopes is not None:
                     s = s - slopes[hd].to(self.cd) * dist
-                o = torch.softmax(s, 0) @ rows[:, g, D:]
+                if softcap:
+                    s = softcap * torch.tanh(s / softcap)
+                if sinks is not None:
+                    s = torch.cat([s, sinks[hd:hd + 1].to(self.cd)])
+                o = torch.softmax(s, 0)[:len(js)] @ rows[:, g, D:]
                 if gate is not None:
                     o = o * torch.sigmoid(
                         gate[t, gate_offset + hd * V:gate_offset + (hd + 1) * V].to(self.cd))
                 out[t, hd * V:(hd + 1) * V] = (o * out_scale).to(out.dtype)
+
+    # -- several copies of the stream -------------------------------------------------------
+    def hyper_mix(self, dst, src, y=None, *, streams, mix=None, write=None, read=None, u=None,
+                  out=None, norm=None):
+        T = src.shape[0]
+        W = (out if out is not None else u if u is not None else y).shape[1]
+        X = src.to(self.cd).view(T, -1, W)
+        X = X.expand(T, streams, W) if X.shape[1] != streams else X
+        if y is not None:
+            X = torch.einsum("st,nsw->ntw", mix.to(self.cd), X) \
+                + write.to(self.cd)[None, :, None] * y.to(self.cd)[:, None, :]
+        if dst is not None:
+            dst.copy_(X.reshape(T, -1).to(dst.dtype))
+        r = torch.ones(streams, dtype=self.cd) if read is None else read.to(self.cd)
+        v = torch.einsum("s,nsw->nw", r, X)
+        if u is not None:
+            u.copy_(v.to(u.dtype))
+        if out is not None:
+            out.copy_((self._rms(v, norm[1]) * norm[0].to(self.cd)).to(out.dtype))
+
+    # -- the state-space recurrence -----------------------------------------------------------
+    def ssm_rows_dtype(self, dtype, n_tokens, sizes):
+        return torch.float32
+
+    @staticmethod
+    def _ssm_split(state, heads, groups, state_dim, vdim, taps):
+        """(states [slots, H, N, V], convolution rings [slots, taps, channels]) of the slots."""
+        n = heads * state_dim * vdim
+        flat = state.view(state.shape[0], -1)
+        return (flat[:, :n].view(-1, heads, state_dim, vdim),
+                flat[:, n:].view(-1, taps, heads * vdim + 2 * groups * state_dim))
+
+    def ssm_prepare(self, rows, step, proj, state, tok_req, tok_pos, req_start, req_slot, *,
+                    conv_w, conv_b, dt_bias, a_log, x_off, heads, groups, state_dim, vdim, taps):
+        _, ring = self._ssm_split(state, heads, groups, state_dim, vdim, taps)
+        C = ring.shape[2]
+        for t in range(rows.shape[0]):
+            r = int(tok_req[t])
+            if r < 0:
+                continue
+            first, pos = int(req_start[r]), int(tok_pos[t])
+            acc = conv_b.to(self.cd).clone()
+            for j in range(taps):
+                back = taps - 1 - j
+                if pos - back < 0:
+                    continue
+                x = proj[t - back, x_off:x_off + C] if t - back >= first \
+                    else ring[int(req_slot[r]), (pos - back) % taps]
+                acc = acc + conv_w[j].to(self.cd) * x.to(self.cd)
+            rows[t] = (acc * torch.sigmoid(acc)).to(rows.dtype)
+            z = proj[t, x_off + C:x_off + C + heads].to(self.cd) + dt_bias.to(self.cd)
+            dt = torch.nn.functional.softplus(z, threshold=1e9)
+            step[t] = torch.cat([dt, -torch.exp(a_log.to(self.cd)) * dt]).to(step.dtype)
+
+    def ssm_recurrence(self, y, state, rows, step, proj, skip, tok_pos, req_start, req_len,
+                       req_slot, *, x_off, heads, groups, state_dim, vdim, taps):
+        H, G, N, V = heads, groups, state_dim, vdim
+        S_all, ring = self._ssm_split(state, H, G, N, V, taps)
+        C = ring.shape[2]
+        for r in range(req_start.shape[0]):
+            n = int(req_len[r])
+            if n <= 0:
+                continue
+            t0, slot = int(req_start[r]), int(req_slot[r])
+            for h in range(H):
+                g = h // (H // G)
+                S = S_all[slot, h].to(self.cd)
+                for t in range(t0, t0 + n):
+                    x = rows[t, h * V:(h + 1) * V].to(self.cd)
+                    B = rows[t, H * V + g * N:H * V + (g + 1) * N].to(self.cd)
+                    Cr = rows[t, H * V + (G + g) * N:H * V + (G + g + 1) * N].to(self.cd)
+                    dt, la = step[t, h].to(self.cd), step[t, H + h].to(self.cd)
+                    S = torch.exp(la) * S + dt * B[:, None] * x[None, :]
+                    y[t, h * V:(h + 1) * V] = (Cr @ S + skip[h].to(self.cd) * x).to(y.dtype)
+                S_all[slot, h] = S.to(state.dtype)
+            for t in range(max(t0, t0 + n - taps), t0 + n):
+                ring[slot, int(tok_pos[t]) % taps] = proj[t, x_off:x_off + C]
+
+    def ssm_step(self, y, state, proj, skip, tok_req, tok_pos, req_slot, *, conv_w, conv_b,
+                 dt_bias, a_log, x_off, heads, groups, state_dim, vdim, taps):
+        T = y.shape[0]
+        sizes = dict(heads=heads, groups=groups, state_dim=state_dim, vdim=vdim, taps=taps)
+        R = req_slot.shape[0]
+        start, length = torch.zeros(R, dtype=torch.int32), torch.zeros(R, dtype=torch.int32)
+        for t in range(T):
+            if int(tok_req[t]) >= 0:
+                start[int(tok_req[t])], length[int(tok_req[t])] = t, 1
+        rows = torch.zeros(T, heads * vdim + 2 * groups * state_dim, dtype=y.dtype)
+        step = torch.zeros(T, 2 * heads, dtype=y.dtype)
+        self.ssm_prepare(rows, step, proj, state, tok_req, tok_pos, start, req_slot, conv_w=conv_w,
+                         conv_b=conv_b, dt_bias=dt_bias, a_log=a_log, x_off=x_off, **sizes)
+        self.ssm_recurrence(y, state, rows, step, proj, skip, tok_pos, start, length, req_slot,
+                            x_off=x_off, **sizes)
 
     def token_shift_mix(self, out, h, mu, state, tok_req, req_start, req_len, req_slot, *,
                         state_offset):
