@@ -1,16 +1,20 @@
-// Grouped softmax attention over the paged cache with a linear bias of the distance and a
-// sliding window that keeps the first tokens, on the CUDA cores.
+// Grouped softmax attention over the paged cache with a linear bias of the distance, a sliding
+// window that keeps the first tokens, capped scores and a sink, on the CUDA cores.
 //
 // The cache keeps one row [key (D) | value (V)] per token and key/value head (pool
 // [pages][kv_heads][page_size][D + V]).
 //
 //   span_prepare    from the float32 projection: q (and k) divided by their root mean square per
-//                   head when asked (no weight), q to a float32 buffer, the row [k | v] straight
+//                   head when asked (no weight), or both over their whole projections (with
+//                   weights), then turned by the token's position on each head's first rot_dims
+//                   numbers (number i pairs with i + rot_dims/2); q to a float32 buffer, the row [k | v] straight
 //                   into the token's page; the values are columns of their own or the keys as
 //                   projected.  A layer that only reads another's rows writes nothing and has
 //                   no key or value columns.
 //   span_attention  a block per (token, query head).  Query i sees j <= i with i - j < window
-//                   (window 0: all) or j < keep_first; score = q . k * scale - slope_h * (i - j);
+//                   (window 0: all) or j < keep_first; score = q . k * scale - slope_h * (i - j),
+//                   then softcap * tanh(score / softcap) when there is a cap; a sink (one logit a
+//                   head, as it stands) enters the denominator alone;
 //                   its eight warps take rounds of 32 keys in turn (a key per lane for the
 //                   scores, a column per lane for the values, four value rows in flight), each
 //                   with a running softmax of its own, joined under one maximum at the end; the
@@ -21,6 +25,7 @@
 // Scores, softmax state and accumulators are float32.  A row's result depends on its own
 // request only: the keys are dealt to the warps in an order fixed by the position.
 #include "common.cuh"
+#include "rotary.cuh"
 
 namespace hs {
 
@@ -33,14 +38,20 @@ span_prepare_kernel(float* __restrict__ q_out, TC* __restrict__ pool,
                     int v_off, const int* __restrict__ table, int max_pages, int num_pages,
                     const int* __restrict__ tok_pos, const int* __restrict__ tok_req, int H, int G,
                     int D, int V, int qk_norm, float eps, int page_size, int writes,
-                    int* __restrict__ status) {
+                    const float* __restrict__ wq, const float* __restrict__ wk,
+                    const float* __restrict__ freq, int rot_dims, int* __restrict__ status) {
+  extern __shared__ float2 s_turn[];               // cosine and sine per turned pair
+  __shared__ float s_sq[2][SA_WARPS];
   pdl_trigger();
-  pdl_wait();
   const int t = blockIdx.x;
   const int r = tok_req[t];
   if (r < 0) return;
   const int pos = tok_pos[t];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int half = rot_dims >> 1;
+  for (int i = threadIdx.x; i < half; i += SA_WARPS * 32)
+    pair_angle(pos, freq[i], &s_turn[i].x, &s_turn[i].y);
+  pdl_wait();
   TC* row = nullptr;
   if (writes) {
     const int pi = pos / page_size;
@@ -52,6 +63,31 @@ span_prepare_kernel(float* __restrict__ q_out, TC* __restrict__ pool,
     }
   }
   const float* pr = proj + (size_t)t * proj_stride;
+  float rq = 1.0f, rk = 1.0f;                      // of the whole projections
+  if (wq) {
+    float sq = 0.f, sk = 0.f;
+    for (int e = threadIdx.x; e < H * D; e += SA_WARPS * 32) sq = fmaf(pr[q_off + e], pr[q_off + e], sq);
+    if (row)
+      for (int e = threadIdx.x; e < G * D; e += SA_WARPS * 32)
+        sk = fmaf(pr[k_off + e], pr[k_off + e], sk);
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) {
+      s_sq[0][warp] = sq;
+      s_sq[1][warp] = sk;
+    }
+  }
+  __syncthreads();                                 // the sums, and the pairs' angles
+  if (wq) {
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < SA_WARPS; ++w) {
+      sq += s_sq[0][w];
+      sk += s_sq[1][w];
+    }
+    rq = 1.0f / sqrtf(sq / (float)(H * D) + eps);
+    rk = 1.0f / sqrtf(sk / (float)(G * D) + eps);
+  }
   const int jobs = row ? H + 2 * G : H;            // query heads, key heads, value heads
   for (int job = warp; job < jobs; job += SA_WARPS) {
     const bool is_q = job < H, is_k = !is_q && job < H + G;
@@ -68,10 +104,25 @@ span_prepare_kernel(float* __restrict__ q_out, TC* __restrict__ pool,
       ss = warp_sum(ss);
       rn = 1.0f / sqrtf(ss / (float)n + eps);
     }
+    const float* wt = nullptr;
+    if (wq && (is_q || is_k)) {
+      rn = is_q ? rq : rk;
+      wt = is_q ? wq + (size_t)job * D : wk + (size_t)g * D;
+    }
+    const int turned = (is_q || is_k) ? rot_dims : 0;
     float* qdst = is_q ? q_out + (size_t)t * H * D + (size_t)job * D : nullptr;
     TC* cdst = is_q ? nullptr : row + (size_t)g * page_size * (D + V) + (is_k ? 0 : D);
     for (int e = lane; e < n; e += 32) {
-      const float val = src[e] * rn;
+      float val = src[e] * rn;
+      if (wt) val *= wt[e];
+      if (e < turned) {
+        const bool low = e < half;
+        const int pe = low ? e + half : e - half;
+        float other = src[pe] * rn;
+        if (wt) other *= wt[pe];
+        const float2 cs = s_turn[low ? e : pe];
+        val = low ? val * cs.x - other * cs.y : val * cs.x + other * cs.y;
+      }
       if (qdst) qdst[e] = val;
       else cdst[e] = from_f<TC>(val);
     }
@@ -125,7 +176,7 @@ span_attention_kernel(TO* __restrict__ out, const float* __restrict__ q,
                       float out_scale, int n_tokens, int H, int G, int D, int V, int window,
                       int keep_first, float scale, int page_size, int vec,
                       const int* __restrict__ listed, const int* __restrict__ plan_head,
-                      int* __restrict__ status) {
+                      float softcap, const float* __restrict__ sinks, int* __restrict__ status) {
   extern __shared__ float s_sa[];                  // q [D] | acc [SA_WARPS][V] | m, l [2 SA_WARPS]
   float* sq = s_sa;
   float* s_acc = s_sa + D;
@@ -170,7 +221,8 @@ span_attention_kernel(TO* __restrict__ out, const float* __restrict__ q,
       else krow = pool + (((size_t)page * G + g) * page_size + (j % page_size)) * (size_t)row_len;
     }
     // the bias of the distance is taken off the scaled score
-    const float s = krow ? sa_dot(krow, sq, D, vec != 0) - slope * (float)(pos - j) : -INFINITY;
+    float s = krow ? sa_dot(krow, sq, D, vec != 0) - slope * (float)(pos - j) : -INFINITY;
+    if (softcap > 0.f && krow) s = softcap * tanhf(s / softcap);
     const float m_new = fmaxf(m, warp_max(s));
     if (m_new == -INFINITY) continue;               // no valid key in this round
     const float corr = expf(m - m_new);             // m = -inf: 0
@@ -222,7 +274,8 @@ span_attention_kernel(TO* __restrict__ out, const float* __restrict__ q,
   float top = -INFINITY;
 #pragma unroll
   for (int w = 0; w < SA_WARPS; ++w) top = fmaxf(top, s_ml[w]);
-  float total = 0.f, share[SA_WARPS];
+  if (sinks) top = fmaxf(top, sinks[h]);
+  float total = sinks ? expf(sinks[h] - top) : 0.f, share[SA_WARPS];
 #pragma unroll
   for (int w = 0; w < SA_WARPS; ++w) {
     share[w] = s_ml[w] == -INFINITY ? 0.f : expf(s_ml[w] - top);
@@ -250,7 +303,8 @@ HS_EXPORT int hs_span_prepare(float* q_out, void* pool, const float* proj, int p
                               int q_off, int k_off, int v_off, const int* table, int max_pages,
                               int num_pages, const int* tok_pos, const int* tok_req,
                               int n_tokens, int H, int G, int D, int V, int qk_norm, float eps,
-                              int page_size, int writes, int cache_dtype, int* status,
+                              int page_size, int writes, const float* wq, const float* wk,
+                              const float* freq, int rot_dims, int cache_dtype, int* status,
                               void* stream) {
   if (!q_out || !pool || !proj || !table || !tok_pos || !tok_req || !status)
     return HS_ERR_ARGUMENT;
@@ -260,19 +314,24 @@ HS_EXPORT int hs_span_prepare(float* q_out, void* pool, const float* proj, int p
   if (writes && (k_off < 0 || k_off + G * D > proj_stride || (v_off < 0 && V != D) ||
                  (v_off >= 0 && v_off + G * V > proj_stride)))
     return HS_ERR_UNSUPPORTED;
+  if (rot_dims < 0 || rot_dims % 2 || rot_dims > D || (rot_dims && !freq) || (wq && qk_norm) ||
+      (wq && writes && !wk))
+    return HS_ERR_ARGUMENT;
   if (n_tokens <= 0) return HS_OK;
+  const size_t smem = (size_t)(rot_dims / 2) * sizeof(float2);
+  if (smem > 40 * 1024) return HS_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
   cudaError_t e;
   if (cache_dtype == HS_DT_BF16)
     e = hs_launch(hs::span_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(hs::SA_WARPS * 32),
-                  0, st, hs_pdl_enabled(), q_out, (__nv_bfloat16*)pool, proj, proj_stride, q_off,
+                  smem, st, hs_pdl_enabled(), q_out, (__nv_bfloat16*)pool, proj, proj_stride, q_off,
                   k_off, v_off, table, max_pages, num_pages, tok_pos, tok_req, H, G, D, V, qk_norm,
-                  eps, page_size, writes, status);
+                  eps, page_size, writes, wq, wk, freq, rot_dims, status);
   else if (cache_dtype == HS_DT_F32)
-    e = hs_launch(hs::span_prepare_kernel<float>, dim3(n_tokens), dim3(hs::SA_WARPS * 32), 0, st,
+    e = hs_launch(hs::span_prepare_kernel<float>, dim3(n_tokens), dim3(hs::SA_WARPS * 32), smem, st,
                   hs_pdl_enabled(), q_out, (float*)pool, proj, proj_stride, q_off, k_off, v_off,
                   table, max_pages, num_pages, tok_pos, tok_req, H, G, D, V, qk_norm, eps,
-                  page_size, writes, status);
+                  page_size, writes, wq, wk, freq, rot_dims, status);
   else
     return HS_ERR_UNSUPPORTED;
   return e == cudaSuccess ? HS_OK : (int)e;
@@ -284,8 +343,8 @@ HS_EXPORT int hs_span_attention(void* out, const float* q, const void* pool, con
                                 int gate_stride, int gate_offset, float out_scale, int n_tokens,
                                 int H, int G, int D, int V, int window, int keep_first,
                                 float scale, int page_size, int cache_dtype, int out_dtype,
-                                const int* listed, const int* plan_head, int* status,
-                                void* stream) {
+                                const int* listed, const int* plan_head, float softcap,
+                                const float* sinks, int* status, void* stream) {
   if (!out || !q || !pool || !table || !tok_pos || !tok_req || !status || (listed && !plan_head))
     return HS_ERR_ARGUMENT;
   if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0 || V > 1024 || window < 0 ||
@@ -308,7 +367,7 @@ HS_EXPORT int hs_span_attention(void* out, const float* q, const void* pool, con
   e = hs_launch(hs::span_attention_kernel<TC, TO, C>, grid, blk, smem, st, pdl, (TO*)out, q,     \
                 (const TC*)pool, table, max_pages, num_pages, tok_pos, tok_req, slopes, gate,    \
                 gate_stride, gate_offset, out_scale, n_tokens, H, G, D, V, window, keep_first,   \
-                scale, page_size, vec, listed, plan_head, status)
+                scale, page_size, vec, listed, plan_head, softcap, sinks, status)
 #define HS_SA_LAUNCH(TC, TO)                                                                     \
   do {                                                                                           \
     if (V <= 64) HS_SA_LAUNCH_C(TC, TO, 2);                                                      \

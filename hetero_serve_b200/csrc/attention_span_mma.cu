@@ -11,7 +11,8 @@
 //     first the kept rows that lie before the window of the item's FIRST query, then the token
 //     rows from that window on (kept rows among them count by the second rule); the two ranges
 //     are apart, so no key counts twice, and a warp skips tiles none of its rows see;
-//   * the score loses slope_h * (i - j), in the accumulators;
+//   * the score loses slope_h * (i - j), in the accumulators, and may then be capped,
+//     cap * tanh(s / cap); a sink may join the denominator at the end;
 //   * the queries arrive in float32 (normed or not) and are rounded once, into shared memory;
 //   * the head's output may be multiplied element by element by the sigmoid of gate columns and
 //     by a scale before it is rounded.
@@ -34,7 +35,8 @@ struct SpanPrefillParams {
   int* work_counter;         // next work item; zero at launch
   int n_heads, n_kv_heads, page_size, num_pages, max_pages;
   int window, keep_first, gate_stride, gate_offset;
-  float scale, out_scale;
+  float scale, out_scale, softcap;
+  const float* sinks;        // [heads] or null
 };
 
 // 16-byte chunks of a row of N numbers, permuted by the row inside groups of 8, 4 or 2 chunks
@@ -105,6 +107,8 @@ span_prefill_kernel(const SpanPrefillParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   const float sc = p.scale * 1.4426950408889634f;        // scores in units of log2(e)
+  const float cap2 = p.softcap * 1.4426950408889634f;
+  const float cap_in = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;   // e^(2 s / cap) as a power of 2
   while (true) {
   __syncthreads();            // the previous item's shared memory has been consumed
   if (threadIdx.x == 0) s_item = atomicAdd(p.work_counter, 1);
@@ -252,7 +256,10 @@ span_prefill_kernel(const SpanPrefillParams p) {
           // as kept first rows.  The two ranges are apart, so no key counts twice.
           const bool sees = mean ? j < (c < 2 ? seen_a : seen_b)
                                  : (j <= i && (j > i - win || j < p.keep_first) && j >= key_lo);
-          s[nt][c] = sees ? fmaf(s[nt][c], sc, -slope * (float)(i - j)) : -INFINITY;
+          float v = fmaf(s[nt][c], sc, -slope * (float)(i - j));
+          if (p.softcap > 0.f)               // cap * tanh(v / cap), both in units of log2(e)
+            v = cap2 * (1.0f - __fdividef(2.0f, 1.0f + exp2f(v * cap_in)));
+          s[nt][c] = sees ? v : -INFINITY;
         }
         mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
         mx_b = fmaxf(mx_b, fmaxf(s[nt][2], s[nt][3]));
@@ -312,6 +319,17 @@ span_prefill_kernel(const SpanPrefillParams p) {
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+  if (p.sinks) {
+    const float sk = p.sinks[h] * 1.4426950408889634f;
+    const float ta = fmaxf(m_a, sk), tb = fmaxf(m_b, sk);
+    const float ea = exp2f(m_a - ta), eb = exp2f(m_b - tb);      // nothing seen: 0
+    l_a = l_a * ea + exp2f(sk - ta);
+    l_b = l_b * eb + exp2f(sk - tb);
+#pragma unroll
+    for (int i = 0; i < DT; ++i) {
+      o[i][0] *= ea; o[i][1] *= ea; o[i][2] *= eb; o[i][3] *= eb;
+    }
+  }
   const float ia = l_a > 0.f ? 1.f / l_a : 0.f, ib = l_b > 0.f ? 1.f / l_b : 0.f;
   __nv_bfloat16* oa = p.out + ((size_t)(tok0 + row_a) * p.n_heads + h) * V;
   __nv_bfloat16* ob = p.out + ((size_t)(tok0 + row_b) * p.n_heads + h) * V;
@@ -371,7 +389,8 @@ HS_EXPORT int hs_span_attention_prefill(void* out, const float* q, const void* p
                                         int gate_stride, int gate_offset, float out_scale,
                                         int n_heads, int n_kv_heads, int head_dim, int value_dim,
                                         int window, int keep_first, float scale, int page_size,
-                                        int* status, void* stream) {
+                                        float softcap, const float* sinks, int* status,
+                                        void* stream) {
   using namespace hs;
   if (!out || !q || !pool || !table || !tile_info || !plan_head || !status || !work_counter)
     return HS_ERR_ARGUMENT;
@@ -387,7 +406,7 @@ HS_EXPORT int hs_span_attention_prefill(void* out, const float* q, const void* p
   p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.page_size = page_size;
   p.num_pages = num_pages; p.max_pages = max_pages; p.window = window;
   p.keep_first = keep_first; p.gate_stride = gate_stride; p.gate_offset = gate_offset;
-  p.scale = scale; p.out_scale = out_scale;
+  p.scale = scale; p.out_scale = out_scale; p.softcap = softcap; p.sinks = sinks;
   cudaStream_t st = (cudaStream_t)stream;
 #define HS_SP_CASE(DD, VV) \
   if (head_dim == DD && value_dim == VV) return launch_span_prefill<DD, VV>(p, st)

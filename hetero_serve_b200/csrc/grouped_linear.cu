@@ -8,12 +8,23 @@
 // tokens x 32 output columns; its four or eight warps (the caller's choice) each sum their part of k for
 // every column, and the parts are added in a fixed order, so a row's result depends on nothing else in the batch.
 //
+// `gate` (may be null): float32 rows; the sum is multiplied by sigmoid(gate[t, gate_off + g * n + j])
+// before it is rounded.
+//
 // `list` (may be null): a step's attention plan; then row i of the launch is the i-th single-query
 // token of the plan (`n_tokens` bounds their number) and no other token is touched.
 #include "common.cuh"
 #include "mma_tiles.cuh"
 
 namespace hs {
+
+struct GlGate {
+  const float* rows;
+  int stride, off;
+  __device__ __forceinline__ float apply(float v, int t, int c) const {
+    return rows ? v / (1.0f + expf(-rows[(size_t)t * stride + off + c])) : v;
+  }
+};
 
 // the token of row i: list = {count, -, -, -, token, -, -, token, ...}
 __device__ __forceinline__ int gl_token(const int* list, int i) { return list ? list[4 + 3 * i] : i; }
@@ -25,7 +36,8 @@ template <typename TW, typename TO, int GL_WARPS>
 __global__ void __launch_bounds__(32 * GL_WARPS)
 grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
                       const TW* __restrict__ w, int n_tokens, int a_stride, int a_off,
-                      int a_gstride, int groups, int n, int k, const int* __restrict__ list) {
+                      int a_gstride, int groups, int n, int k, const int* __restrict__ list,
+                      const GlGate gate) {
   extern __shared__ float s_a[];                    // [GL_TT][k]
   pdl_trigger();
   pdl_wait();
@@ -70,7 +82,8 @@ grouped_linear_kernel(TO* __restrict__ out, const float* __restrict__ a,
       float v = s_part[0][tt][c];
 #pragma unroll
       for (int q = 1; q < GL_WARPS; ++q) v += s_part[q][tt][c];
-      out[(size_t)gl_token(list, t0 + tt) * groups * n + (size_t)g * n + col] = from_f<TO>(v);
+      const int t = gl_token(list, t0 + tt);
+      out[(size_t)t * groups * n + (size_t)g * n + col] = from_f<TO>(gate.apply(v, t, g * n + col));
     }
   }
 }
@@ -89,7 +102,7 @@ __global__ void __launch_bounds__(128)
 grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
                           const __nv_bfloat16* __restrict__ w, int n_tokens, int a_stride,
                           int a_off, int a_gstride, int groups, int N, int K, int vec,
-                          const int* __restrict__ list) {
+                          const int* __restrict__ list, const GlGate gate) {
   __shared__ __align__(16) __nv_bfloat16 s_a[2][SPLIT][TM * TS];
   __shared__ __align__(16) __nv_bfloat16 s_b[2][TN * TS];
   pdl_trigger();
@@ -204,9 +217,11 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
 #pragma unroll
         for (int q = 0; q < 2; ++q) {
           const int c = wn + 8 * j + 2 * tq + q;
-          if (c < ncols)
-            out[(size_t)gl_token(list, t0 + r) * groups * N + (size_t)g * N + n0 + c] =
-                from_f<TO>(acc[i][j][2 * half + q]);
+          if (c < ncols) {
+            const int t = gl_token(list, t0 + r);
+            out[(size_t)t * groups * N + (size_t)g * N + n0 + c] =
+                from_f<TO>(gate.apply(acc[i][j][2 * half + q], t, g * N + n0 + c));
+          }
         }
       }
 }
@@ -216,8 +231,10 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const float* __restrict__ a,
 HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_tokens,
                                 int a_stride, int a_off, int a_gstride, int groups, int n, int k,
                                 int w_dtype, int out_dtype, const int* list, int parts,
-                                void* stream) {
+                                const float* gate, int gate_stride, int gate_off, void* stream) {
   if (!out || !a || !w || (parts != 4 && parts != 8)) return HS_ERR_ARGUMENT;
+  if (gate && (gate_off < 0 || gate_off + groups * n > gate_stride)) return HS_ERR_ARGUMENT;
+  const hs::GlGate gt = {gate, gate_stride, gate_off};
   if (groups <= 0 || n <= 0 || k <= 0) return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
   const size_t smem = (size_t)hs::GL_TT * k * sizeof(float);
@@ -231,7 +248,7 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
     if (smem > 32 * 1024)  /* with the static array a block may then pass 48 KB */            \
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     e = hs_launch(kern, grid, dim3(32 * NW), smem, st, hs_pdl_enabled(), (TO*)out, a,         \
-                  (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, list);    \
+                  (const TW*)w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, list, gt); \
   } while (0)
 #define HS_GL(TW, TO)                                                                         \
   do {                                                                                        \
@@ -252,8 +269,11 @@ HS_EXPORT int hs_grouped_linear(void* out, const float* a, const void* w, int n_
 HS_EXPORT int hs_grouped_linear_mma(void* out, const float* a, const void* w_nk, int n_tokens,
                                     int a_stride, int a_off, int a_gstride, int groups, int n,
                                     int k, int out_dtype, int split, const int* list,
+                                    const float* gate, int gate_stride, int gate_off,
                                     void* stream) {
   if (!out || !a || !w_nk) return HS_ERR_ARGUMENT;
+  if (gate && (gate_off < 0 || gate_off + groups * n > gate_stride)) return HS_ERR_ARGUMENT;
+  const hs::GlGate gt = {gate, gate_stride, gate_off};
   if (groups <= 0 || n <= 0 || k <= 0 || k % hs::TK || (split != 1 && split != 3))
     return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
@@ -265,16 +285,16 @@ HS_EXPORT int hs_grouped_linear_mma(void* out, const float* a, const void* w_nk,
   cudaError_t e = cudaSuccess;
   if (out_dtype == HS_DT_F32 && split == 3)
     e = hs_launch(hs::grouped_linear_mma_kernel<float, 3>, grid, dim3(128), 0, st, pdl, (float*)out,
-                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec, list);
+                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec, list, gt);
   else if (split == 3)
     return HS_ERR_UNSUPPORTED;
   else if (out_dtype == HS_DT_F32)
     e = hs_launch(hs::grouped_linear_mma_kernel<float, 1>, grid, dim3(128), 0, st, pdl, (float*)out,
-                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec, list);
+                  a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k, vec, list, gt);
   else if (out_dtype == HS_DT_BF16)
     e = hs_launch(hs::grouped_linear_mma_kernel<__nv_bfloat16, 1>, grid, dim3(128), 0, st, pdl,
                   (__nv_bfloat16*)out, a, w, n_tokens, a_stride, a_off, a_gstride, groups, n, k,
-                  vec, list);
+                  vec, list, gt);
   else
     return HS_ERR_UNSUPPORTED;
   return e == cudaSuccess ? HS_OK : (int)e;

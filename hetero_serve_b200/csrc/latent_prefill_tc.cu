@@ -1,4 +1,4 @@
-// Windowed attention over a shared latent for prompt portions, on tcgen05 tensor cores (sm_100a),
+// Attention over a shared latent for prompt portions, with or without a window, on tcgen05 tensor cores (sm_100a),
 // bfloat16 operands, float32 accumulators.  Same mathematics as latent_attention.cu, in the form
 // that costs prompts least: keys and values are EXPANDED per head, once for every position the
 // step's portions can see, instead of absorbing the expansions into the queries (a query and key
@@ -8,12 +8,14 @@
 //            their pages into a dense block (latents and key parts apart), and the portion's
 //            queries are turned, rounded and padded to whole 64-number chunks, in one launch;
 //   (linear  the dense latents times [W_uk; W_uv], the framework's own product)
-//   attend   S = [q | q_rot] [k | k_rot]^T,  softmax over the window,  O = P V.
+//   attend   S = [q | q_rot] [k | k_rot]^T,  softmax over what is visible,  O = P V, optionally times
+//            the sigmoid of gate columns.
 //
 // Dense rows: position p of request r lies in row base[r] + p.  A portion of n tokens from position
 // s sees positions lo = max(0, s - window + 1) .. s + n - 1; with k requests that bring portions
-// before r, its rows start at req_start[r] + k * (window - 1).  Rows nobody wrote hold zeros or an
-// earlier step's numbers: finite, and always masked.
+// before r, its rows start at req_start[r] + k * (window - 1).  Without a window (0) it sees all
+// positions 0 .. s + n - 1 and its rows follow those of the portions before r.  Rows nobody wrote
+// hold zeros or an earlier step's numbers: finite, and always masked.
 //
 // A block works on up to 128 consecutive queries of one request x one head, 128 keys a tile:
 //   warp 0      TMA producer: the queries once; per tile the key chunks of 64 numbers (the head's
@@ -62,11 +64,18 @@ latent_gather_kernel(__nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict_
       if (part == 0 && threadIdx.x == 0) base[r] = -1;
       return;
     }
-    int before = 0;
-    for (int i = 0; i < r; ++i) before += req_len[i] > max_single;
     const int pos0 = tok_pos[req_start[r]];
-    const int lo = max(0, pos0 + 1 - window), rows = pos0 + n - lo;
-    const int row0 = req_start[r] + before * (window - 1);
+    int lo = 0, row0 = 0;
+    if (window > 0) {
+      int before = 0;
+      for (int i = 0; i < r; ++i) before += req_len[i] > max_single;
+      lo = max(0, pos0 + 1 - window);
+      row0 = req_start[r] + before * (window - 1);
+    } else {
+      for (int i = 0; i < r; ++i)
+        if (req_len[i] > max_single) row0 += tok_pos[req_start[i]] + req_len[i];
+    }
+    const int rows = pos0 + n - lo;
     if (part == 0 && threadIdx.x == 0) base[r] = row0 - lo;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int W = R + P;
@@ -133,8 +142,10 @@ struct LatentTcParams {
   const int* plan;
   const int* base;
   int* status;
-  int tiles_off, n_heads, D, V, window, cap_rows;
+  int tiles_off, n_heads, D, V, window, cap_rows;     // window: huge when there is none
   float scale;
+  const float* gate;              // [tokens, gate_stride] or null: column gate_off + h * V + e
+  int gate_stride, gate_off;
 };
 
 enum { LB_Q = 0, LB_K_FULL = 1, LB_K_EMPTY = 3, LB_V_FULL = 5, LB_V_EMPTY = 6, LB_S_FULL = 7,
@@ -392,14 +403,22 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (ok && row < nq) {
       const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
       __nv_bfloat16* orow = p.out + ((size_t)(tok0 + row) * p.n_heads + h) * p.V;
+      const float* grow = p.gate ? p.gate + (size_t)(tok0 + row) * p.gate_stride + p.gate_off +
+                                       (size_t)h * p.V + half * OC
+                                 : nullptr;
       // this thread's columns are half * OC .. + OC - 1; V is a multiple of 8
 #pragma unroll
       for (int c = 0; c < OC; c += 8) {
         if (half * OC + c >= p.V) continue;
         uint32_t u[4];
+        float w[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          w[i] = grow ? __fdividef(inv, 1.0f + __expf(-grow[c + i])) : inv;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          const __nv_bfloat162 b2 = __floats2bfloat162_rn(o[c + 2 * i] * inv, o[c + 2 * i + 1] * inv);
+          const __nv_bfloat162 b2 =
+              __floats2bfloat162_rn(o[c + 2 * i] * w[2 * i], o[c + 2 * i + 1] * w[2 * i + 1]);
           u[i] = *(const uint32_t*)&b2;
         }
         *(uint4*)(orow + half * OC + c) = make_uint4(u[0], u[1], u[2], u[3]);
@@ -447,26 +466,28 @@ static int lp_map(CUtensorMap* map, const void* base, long long rows, long long 
 // 128 + 64 numbers, values of up to 128.
 HS_EXPORT int hs_latent_prefill_tc_takes(int D, int P, int V, int R, int window, float scale) {
   return D > 0 && D <= 128 && D % 8 == 0 && P > 0 && P <= 64 && V > 0 && V <= 128 && V % 8 == 0 &&
-                 R > 0 && R % 8 == 0 && window > 0 && scale > 0.f
+                 R > 0 && R % 8 == 0 && window >= 0 && scale > 0.f
              ? 1
              : 0;
 }
 
 // lat [cap_rows, R], rope [cap_rows, 64], q_out [n_tokens, n_heads * (pad64(D) + 64)], base
-// [n_requests]; q [n_tokens, n_heads * (D + P)] float32.  Requests of up to max_single tokens are
+// [n_requests]; q [n_tokens, n_heads * (D + P)] float32, rows q_stride numbers apart.  Requests of up to max_single tokens are
 // not gathered (their base is -1).
 HS_EXPORT int hs_latent_gather(void* lat, void* rope, void* q_out, int* base, const float* q,
                                const void* pool, const int* table, const int* req_start,
                                const int* req_len, const int* tok_pos, const int* tok_req,
                                int n_requests, int n_tokens, int cap_rows, int window,
-                               int max_single, int R, int P, int n_heads, int D, int page_size,
+                               int max_single, int R, int P, int n_heads, int D, int q_stride,
+                               int page_size,
                                int num_pages, int max_pages, const float* freq, int rot_dims,
                                int* status, void* stream) {
   if (!lat || !rope || !q_out || !base || !q || !pool || !table || !req_start || !req_len ||
       !tok_pos || !tok_req || !status)
     return HS_ERR_ARGUMENT;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > P || (rot_dims && !freq)) return HS_ERR_ARGUMENT;
-  if (window <= 0 || R <= 0 || P <= 0 || P > 64 || D <= 0 || D % 2 || n_heads <= 0 || page_size <= 0)
+  if (window < 0 || R <= 0 || P <= 0 || P > 64 || D <= 0 || D % 2 || n_heads <= 0 ||
+      page_size <= 0 || q_stride < n_heads * (D + P))
     return HS_ERR_UNSUPPORTED;
   if (n_requests <= 0 || n_tokens <= 0) return HS_OK;
   const int pad = (D + 63) / 64 * 64;
@@ -475,7 +496,7 @@ HS_EXPORT int hs_latent_gather(void* lat, void* rope, void* q_out, int* base, co
       (cudaStream_t)stream, hs_pdl_enabled(), (__nv_bfloat16*)lat, (__nv_bfloat16*)rope,
       (__nv_bfloat16*)q_out, base, q, (const __nv_bfloat16*)pool, table, req_start, req_len,
       tok_pos, tok_req, n_requests, n_tokens, cap_rows, window, max_single, R, P, n_heads, D, pad,
-      n_heads * (D + P), page_size, num_pages, max_pages, freq, rot_dims, status);
+      q_stride, page_size, num_pages, max_pages, freq, rot_dims, status);
   return e == cudaSuccess ? HS_OK : (int)e;
 }
 
@@ -483,8 +504,10 @@ HS_EXPORT int hs_latent_gather(void* lat, void* rope, void* q_out, int* base, co
 HS_EXPORT int hs_latent_prefill_tc(void* out, const void* q, const void* kv, const void* rope,
                                    const int* base, const int* plan, int tiles_off, int tile_cap,
                                    int n_tokens, int cap_rows, int n_heads, int D, int P, int V,
-                                   int R, int window, float scale, int* status, void* stream) {
+                                   int R, int window, float scale, const float* gate,
+                                   int gate_stride, int gate_off, int* status, void* stream) {
   using namespace hs;
+  if (gate && (gate_off < 0 || gate_off + n_heads * V > gate_stride)) return HS_ERR_ARGUMENT;
   if (!out || !q || !kv || !rope || !base || !plan || !status) return HS_ERR_ARGUMENT;
   if (!hs_latent_prefill_tc_takes(D, P, V, R, window, scale) || n_heads <= 0)
     return HS_ERR_UNSUPPORTED;
@@ -497,7 +520,9 @@ HS_EXPORT int hs_latent_prefill_tc(void* out, const void* q, const void* kv, con
   if (int e = lp_map(&mr, rope, cap_rows, 64)) return e;
   LatentTcParams p;
   p.out = (__nv_bfloat16*)out; p.plan = plan; p.base = base; p.status = status;
-  p.tiles_off = tiles_off; p.n_heads = n_heads; p.D = D; p.V = V; p.window = window;
+  p.tiles_off = tiles_off; p.n_heads = n_heads; p.D = D; p.V = V;
+  p.window = window > 0 ? window : 1 << 28;
+  p.gate = gate; p.gate_stride = gate_stride; p.gate_off = gate_off;
   p.cap_rows = cap_rows; p.scale = scale;
   const dim3 grid(n_heads, tile_cap), block(LP_THREADS);
   cudaError_t e = cudaSuccess;

@@ -1,5 +1,5 @@
-// The residual stream at the two places where a parallel block touches it, each with the layer
-// norm of what comes next in the same launch:
+// The residual stream at the places where blocks touch it, each with the norm of what comes next in
+// the same launch:
 //
 //   embed_norm     x  = norm(table[id])                            (weight, optional bias)
 //                  x0 = x                                          (optional copy, kept for `again`)
@@ -7,7 +7,11 @@
 //
 //   then, optional in both:  out = norm2(x), float32 or bfloat16
 //
-// The norms are (v - mean) / sqrt(variance + eps) * weight (+ bias), the variance being the mean of
+//   hyper_mix      several copies of the stream behind a sublayer (a token's copies are neighbours
+//                  in one row):  x_t <- sum_s mix[s][t] x_s + write[t] y;
+//                  u = sum_t read[t] x_t;  out = u / sqrt(mean(u^2) + eps) * weight
+//
+// The norms of the first two are (v - mean) / sqrt(variance + eps) * weight (+ bias), the variance being the mean of
 // the squared deviations.  One block per row.  All sums are float32, formed in an order fixed by
 // the width, so a row's result does not depend on its neighbours in the batch.
 #include "common.cuh"
@@ -170,6 +174,90 @@ embed_norm_kernel(float* __restrict__ x, float* __restrict__ x0, const int* __re
   if (out) row_norm_out<VEC>(row, out + at, g2, b2, eps2, s_part);
 }
 
+constexpr int HM_MAX = 16;            // copies of the stream at most
+
+// SM: copies a thread holds (exactly n_streams for SM <= 4).  src holds src_streams rows a token, or
+// one row that stands for all copies; dst may be src.  y, dst, u, out may be null; without y the
+// copies stay as they are; without rd every copy counts once in u.
+template <bool VEC, int SM, typename TO>
+__global__ void __launch_bounds__(SM_THREADS)
+hyper_mix_kernel(float* dst, const float* src, int src_streams, const float* __restrict__ y,
+                 int n_streams, const float* __restrict__ mix, const float* __restrict__ wr,
+                 const float* __restrict__ rd, int width, float* __restrict__ u,
+                 TO* __restrict__ out, const float* __restrict__ g, float eps) {
+  extern __shared__ __align__(16) float s_row[];
+  __shared__ float s_part[SM_THREADS / 32];
+  __shared__ float s_mix[HM_MAX * HM_MAX], s_wr[HM_MAX], s_rd[HM_MAX];
+  pdl_trigger();
+  const int n = SM <= 4 ? SM : n_streams;
+  // the tables are weights: fetched ahead of the wait
+  if (y)
+    for (int i = threadIdx.x; i < n * n; i += blockDim.x) s_mix[i] = mix[i];
+  if ((int)threadIdx.x < n) {
+    s_wr[threadIdx.x] = y ? wr[threadIdx.x] : 0.f;
+    s_rd[threadIdx.x] = rd ? rd[threadIdx.x] : 1.f;
+  }
+  __syncthreads();
+  pdl_wait();
+  Row<VEC> row;
+  row.s = s_row;
+  row.width = width;
+  const size_t t = blockIdx.x;
+  const float* sr = src + t * src_streams * width;
+  const size_t step = src_streams > 1 ? width : 0;
+  float* dr = dst ? dst + t * n * width : nullptr;
+  row.each([&](int c, float* d) {
+    __align__(16) float xs[SM][PIECE<VEC>], yv[PIECE<VEC>], acc[PIECE<VEC>];
+#pragma unroll
+    for (int s = 0; s < SM; ++s)
+      if (s < n) load_piece<VEC>(xs[s], sr + s * step + c);
+#pragma unroll
+    for (int i = 0; i < PIECE<VEC>; ++i) acc[i] = 0.f;
+    if (y) load_piece<VEC>(yv, y + t * width + c);
+#pragma unroll
+    for (int to = 0; to < SM; ++to) {
+      if (to >= n) continue;
+      __align__(16) float v[PIECE<VEC>];
+      if (y) {
+        const float w = s_wr[to];
+#pragma unroll
+        for (int i = 0; i < PIECE<VEC>; ++i) v[i] = w * yv[i];
+#pragma unroll
+        for (int s = 0; s < SM; ++s) {
+          if (s >= n) continue;
+          const float m = s_mix[s * n + to];
+#pragma unroll
+          for (int i = 0; i < PIECE<VEC>; ++i) v[i] = fmaf(m, xs[s][i], v[i]);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < PIECE<VEC>; ++i) v[i] = xs[to][i];
+      }
+      if (dr) store_piece<VEC>(dr + (size_t)to * width + c, v);
+      const float r = s_rd[to];
+#pragma unroll
+      for (int i = 0; i < PIECE<VEC>; ++i) acc[i] = fmaf(r, v[i], acc[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < PIECE<VEC>; ++i) d[i] = acc[i];
+    if (u) store_piece<VEC>(u + t * width + c, d);
+  });
+  if (!out) return;
+  float q = 0.f;
+  row.each([&](int, float* d) {
+#pragma unroll
+    for (int i = 0; i < PIECE<VEC>; ++i) q = fmaf(d[i], d[i], q);
+  });
+  const float r = 1.0f / sqrtf(sm_block_sum(q, s_part) / (float)width + eps);
+  row.each([&](int c, float* d) {
+    __align__(16) float o[PIECE<VEC>], w[PIECE<VEC>];
+    load_piece<VEC>(w, g + c);
+#pragma unroll
+    for (int i = 0; i < PIECE<VEC>; ++i) o[i] = d[i] * r * w[i];
+    store_piece<VEC>(out + t * width + c, o);
+  });
+}
+
 template <bool VEC, typename TO>
 __global__ void __launch_bounds__(SM_THREADS)
 residual_mix_kernel(float* __restrict__ x, const float* __restrict__ y1,
@@ -285,5 +373,43 @@ HS_EXPORT int hs_residual_mix(float* x, const float* y1, const float* s1, const 
   else if (!out || out_dtype == HS_DT_F32) { if (vec) HS_RM(true, float); else HS_RM(false, float); }
   else return HS_ERR_UNSUPPORTED;
 #undef HS_RM
+  return e == cudaSuccess ? HS_OK : (int)e;
+}
+
+// See hyper_mix_kernel.  src_streams: 1 or n_streams rows a token in src.
+HS_EXPORT int hs_hyper_mix(float* dst, const float* src, int src_streams, const float* y,
+                           int n_streams, const float* mix, const float* wr, const float* rd,
+                           int n_rows, int width, float* u, void* out, const float* g, float eps,
+                           int out_dtype, void* stream) {
+  if (!src || (y && (!mix || !wr)) || (!dst && !u && !out) || (out && !g)) return HS_ERR_ARGUMENT;
+  if (width <= 0 || n_streams <= 0 || n_streams > hs::HM_MAX ||
+      (src_streams != 1 && src_streams != n_streams))
+    return HS_ERR_UNSUPPORTED;
+  if (n_rows <= 0) return HS_OK;
+  const void* ptrs[] = {dst, src, y, u, out, g};
+  const bool vec = hs::sm_vec(width, ptrs, 6);
+  const size_t smem = vec ? 0 : (size_t)width * sizeof(float);
+  if (smem > 40 * 1024) return HS_ERR_UNSUPPORTED;
+  const dim3 grid(n_rows), block(hs::sm_threads(width, vec));
+  cudaStream_t st = (cudaStream_t)stream;
+  cudaError_t e = cudaSuccess;
+#define HS_HM(VEC, SM, TO)                                                                      \
+  e = hs_launch(hs::hyper_mix_kernel<VEC, SM, TO>, grid, block, smem, st, hs_pdl_enabled(), dst, \
+                src, src_streams, y, n_streams, mix, wr, rd, width, u, (TO*)out, g, eps)
+#define HS_HM_S(VEC, TO)                      \
+  do {                                        \
+    switch (n_streams) {                      \
+      case 1: HS_HM(VEC, 1, TO); break;       \
+      case 2: HS_HM(VEC, 2, TO); break;       \
+      case 3: HS_HM(VEC, 3, TO); break;       \
+      case 4: HS_HM(VEC, 4, TO); break;       \
+      default: HS_HM(VEC, hs::HM_MAX, TO);    \
+    }                                         \
+  } while (0)
+  if (out && out_dtype == HS_DT_BF16) { if (vec) HS_HM_S(true, __nv_bfloat16); else HS_HM_S(false, __nv_bfloat16); }
+  else if (!out || out_dtype == HS_DT_F32) { if (vec) HS_HM_S(true, float); else HS_HM_S(false, float); }
+  else return HS_ERR_UNSUPPORTED;
+#undef HS_HM_S
+#undef HS_HM
   return e == cudaSuccess ? HS_OK : (int)e;
 }

@@ -253,6 +253,41 @@ timemix_kernel(float* __restrict__ o, float* __restrict__ state, int state_strid
 }
 
 // ---------------------------------------------------------------------------------------
+// a block per (token, part of the row): o times its gate, then the part's root mean square, weight,
+// scale.  The products stay in shared memory between the two.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+gated_part_norm_kernel(TO* __restrict__ out, const float* __restrict__ o,
+                       const float* __restrict__ weight, const float* __restrict__ gate,
+                       int gate_stride, int gate_offset, int H, int D, float eps, int silu,
+                       float out_scale) {
+  extern __shared__ float s_gp[];                       // [D]
+  __shared__ float s_sum[8];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x / H, h = blockIdx.x - t * H;
+  const size_t at = (size_t)t * H * D + (size_t)h * D;
+  const float* g = gate + (size_t)t * gate_stride + gate_offset + (size_t)h * D;
+  float ss = 0.f;
+#pragma unroll 4
+  for (int e = threadIdx.x; e < D; e += blockDim.x) {
+    const float z = g[e], s = 1.0f / (1.0f + expf(-z));
+    const float v = o[at + e] * (silu ? z * s : s);
+    s_gp[e] = v;                                        // read back below by this thread alone
+    ss = fmaf(v, v, ss);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) s_sum[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float total = 0.f;
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) total += s_sum[i];
+  const float r = 1.0f / sqrtf(total / (float)D + eps);
+#pragma unroll 4
+  for (int e = threadIdx.x; e < D; e += blockDim.x)
+    out[at + e] = from_f<TO>(s_gp[e] * r * (weight ? weight[(size_t)h * D + e] : 1.0f) * out_scale);
+}
+
+// ---------------------------------------------------------------------------------------
 // a warp per (token, head): the head's rows of o, its root mean square, weight, gate, scale
 template <typename TO>
 __global__ void __launch_bounds__(256)
@@ -372,8 +407,8 @@ HS_EXPORT int hs_timemix_recurrence(float* o, float* state, int state_stride, co
 HS_EXPORT int hs_head_norm_gate(void* out, const float* o, const float* weight,
                                 const float* gate, int gate_stride, int gate_offset,
                                 int n_tokens, int H, int D, float eps, int gate_silu,
-                                float out_scale, int out_dtype, void* stream) {
-  if (!out || !o) return HS_ERR_ARGUMENT;
+                                float out_scale, int gate_first, int out_dtype, void* stream) {
+  if (!out || !o || (gate_first && !gate)) return HS_ERR_ARGUMENT;
   if (H <= 0 || D <= 0 || (gate && (gate_offset < 0 || gate_offset + H * D > gate_stride)))
     return HS_ERR_UNSUPPORTED;
   if (n_tokens <= 0) return HS_OK;
@@ -381,6 +416,23 @@ HS_EXPORT int hs_head_norm_gate(void* out, const float* o, const float* weight,
   const unsigned blocks = (unsigned)((items + 7) / 8);
   cudaStream_t st = (cudaStream_t)stream;
   cudaError_t e;
+  if (gate_first) {
+    const size_t smem = (size_t)D * sizeof(float);
+    if (smem > 47 * 1024) return HS_ERR_UNSUPPORTED;
+    if (items > 0x7fffffffLL) return HS_ERR_TOO_LARGE;
+    const int threads = D >= 256 ? 256 : (D + 31) / 32 * 32;
+    if (out_dtype == HS_DT_F32)
+      e = hs_launch(hs::gated_part_norm_kernel<float>, dim3((unsigned)items), dim3(threads), smem, st,
+                    hs_pdl_enabled(), (float*)out, o, weight, gate, gate_stride, gate_offset, H, D,
+                    eps, gate_silu, out_scale);
+    else if (out_dtype == HS_DT_BF16)
+      e = hs_launch(hs::gated_part_norm_kernel<__nv_bfloat16>, dim3((unsigned)items), dim3(threads),
+                    smem, st, hs_pdl_enabled(), (__nv_bfloat16*)out, o, weight, gate, gate_stride,
+                    gate_offset, H, D, eps, gate_silu, out_scale);
+    else
+      return HS_ERR_UNSUPPORTED;
+    return e == cudaSuccess ? HS_OK : (int)e;
+  }
   if (out_dtype == HS_DT_F32)
     e = hs_launch(hs::head_norm_gate_kernel<float>, dim3(blocks), dim3(256), 0, st,
                   hs_pdl_enabled(), (float*)out, o, weight, gate, gate_stride, gate_offset,

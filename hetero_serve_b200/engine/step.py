@@ -492,6 +492,8 @@ class Runner:
         if lay.plan_ints:
             plan_shape = self.ops.plan_attention(hm[lay.plan:lay.plan + lay.plan_ints],
                                                  host_batch, T, R, mgr.page_size, self.use_graphs)
+            if self.model.counts_prompt_rows:
+                plan_shape += (self.ops.plan_prompt_rows(host_batch, self.use_graphs),)
 
         # ---- device side -------------------------------------------------------------
         greedy = all(e.temperature <= 0.0 for e in entries)

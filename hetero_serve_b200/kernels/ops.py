@@ -79,6 +79,8 @@ class AttentionPlan:
     decode_cap: int
     tile_cap: int
     single_new: bool = False     # every single-query token is the only new token of its request
+    prompt_rows: int = 0         # at least the positions up to the last token of every request that
+    #                              brings tiles (0: not counted; only some models' parts ask for it)
 
     @property
     def tile_slots(self) -> int:
@@ -200,12 +202,12 @@ def _declare(lib) -> None:
         "hs_dyt_norm": [P, P, P, P, P, I, I, F, I, P],
         "hs_scale": [P, ctypes.c_longlong, F, P],
         "hs_rotary_pairs": [P, P, P, P, I, I, I, I, I, I, P],
-        "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P, I, P],
-        "hs_grouped_linear_mma": [P, P, P, I, I, I, I, I, I, I, I, I, P, P],
+        "hs_grouped_linear": [P, P, P, I, I, I, I, I, I, I, I, I, P, I, P, I, I, P],
+        "hs_grouped_linear_mma": [P, P, P, I, I, I, I, I, I, I, I, I, P, P, I, I, P],
         "hs_latent_decode_mma": [P] * 7 + [I] * 7 + [F, I, I, I, P, P, I, I, P],
         "hs_latent_prefill_tc_takes": [I, I, I, I, I, F],
-        "hs_latent_gather": [P] * 11 + [I] * 12 + [P, I, P, P],
-        "hs_latent_prefill_tc": [P] * 6 + [I] * 10 + [F, P, P],
+        "hs_latent_gather": [P] * 11 + [I] * 13 + [P, I, P, P],
+        "hs_latent_prefill_tc": [P] * 6 + [I] * 10 + [F, P, I, I, P, P],
         "hs_latent_append": [P, P, P, P, P, P, I, I, I, I, I, F, I, I, I, I, P, P, I, P, P, I, I,
                              P],
         "hs_latent_attention": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, P, I,
@@ -233,14 +235,19 @@ def _declare(lib) -> None:
         "hs_token_shift_mix": [P, P, P, P, I, I, P, P, P, P, I, I, I, I, P],
         "hs_timemix_decay": [P, P, P, P, I, I, I, P],
         "hs_timemix_recurrence": [P, P, I, P, P, P, P, P, P, P, P, I, I, I, I, P],
-        "hs_head_norm_gate": [P, P, P, P, I, I, I, I, I, F, I, F, I, P],
+        "hs_head_norm_gate": [P, P, P, P, I, I, I, I, I, F, I, F, I, I, P],
         "hs_gather_mul": [P, P, P, I, I, P, P, P, I, I, I, I, I, I, P, P],
         "hs_moe_route_table": [P, P, P, I, P, P, P, I, I, I, I, P, P],
-        "hs_span_prepare": [P, P, P, I, I, I, I, P, I, I, P, P, I, I, I, I, I, I, F, I, I, I, P, P],
+        "hs_span_prepare": [P, P, P, I, I, I, I, P, I, I, P, P, I, I, I, I, I, I, F, I, I, P, P, P, I,
+                            I, P, P],
         "hs_span_attention": [P, P, P, P, I, I, P, P, P, P, I, I, F, I, I, I, I, I, I, I, F, I, I,
-                              I, P, P, P, P],
+                              I, P, P, F, P, P, P],
         "hs_span_attention_prefill": [P, P, P, P, I, I, P, P, I, P, P, P, I, I, F, I, I, I, I, I, I,
-                                      F, I, P, P],
+                                      F, I, F, P, P, P],
+        "hs_hyper_mix": [P, P, I, P, I, P, P, P, I, I, P, P, P, F, I, P],
+        "hs_ssm_prepare": [P] * 12 + [I] * 10 + [P],
+        "hs_ssm_recurrence": [P] * 10 + [I] * 9 + [P],
+        "hs_ssm_step": [P] * 11 + [I] * 9 + [P],
         "hs_embed_norm": [P, P, P, P, P, I, I, I, I, P, I, P, P, F, P, P, P, F, I, P, P],
         "hs_residual_mix": [P, P, P, P, P, P, I, I, P, P, P, F, I, P],
         "hs_layernorm_add": [P, P, P, P, F, P, P, P, F, I, I, I, P],
@@ -749,6 +756,12 @@ class CudaOps:
                     single)
         return n_dec, n_tiles, single
 
+    @staticmethod
+    def plan_prompt_rows(host_batch, bucketed: bool) -> int:
+        """``AttentionPlan.prompt_rows`` of a batch as ``plan_attention`` takes it."""
+        rows = sum(start + n for _req, _slot, start, n in host_batch if n > DECODE_MAX_NEW)
+        return size_class(rows) if rows and bucketed else rows
+
     def make_plan(self, host_batch, n_rows: int, page_size: int) -> AttentionPlan:
         """A plan built and uploaded on the spot (the runner packs it into the step's single
         upload instead)."""
@@ -756,7 +769,8 @@ class CudaOps:
         view = np.zeros(self.attention_plan_ints(n_rows, len(host_batch)), dtype=np.int32)
         dec, tiles, single = self.plan_attention(view, host_batch, n_rows, len(host_batch),
                                                  page_size, False)
-        return AttentionPlan(torch.from_numpy(view).to(self.device), n_rows, dec, tiles, single)
+        return AttentionPlan(torch.from_numpy(view).to(self.device), n_rows, dec, tiles, single,
+                             self.plan_prompt_rows(host_batch, False))
 
     def _scratch_buffer(self, name, numel, dtype):
         key = (name, dtype)
@@ -1068,7 +1082,7 @@ class CudaOps:
                "rotary_pairs")
 
     def grouped_linear(self, out, a, w, *, a_offset=0, a_group_stride=None, w_nk=None,
-                       exact=False, singles=None, parts=4):
+                       exact=False, singles=None, parts=4, gate=None, gate_offset=0):
         """Block-diagonal linear: ``out[t, g*n + j] = sum_k a[t, a_offset + g*a_group_stride + k]
         * w[g, k, j]``.  ``a`` float32 (a group's input may be a slice of a wider row), ``w``
         [groups, k, n] (k-major), ``out`` [T, groups * n] float32 or of w's type.  ``w_nk`` is
@@ -1078,7 +1092,9 @@ class CudaOps:
         float32: for weights that are bfloat16 numbers the result is then the float32 product,
         and ``out`` is float32).  With ``singles`` (the step's attention plan) only the plan's
         single-query tokens are worked on.  ``parts`` (4 or 8): in how many pieces the CUDA-core
-        kernel cuts the summed index of a few tokens' rows (the order of its additions)."""
+        kernel cuts the summed index of a few tokens' rows (the order of its additions).  With
+        ``gate`` (float32 [T, *]) the result is multiplied by sigmoid(gate[t, gate_offset + g*n +
+        j]) before it is rounded."""
         _want(a, "a", torch.float32, 2)
         _want(w, "w", _FLOATS, 3)
         _want(out, "out", _FLOATS, 2)
@@ -1091,6 +1107,12 @@ class CudaOps:
             raise KernelError("grouped_linear: the groups' inputs exceed a's row")
         if out.dtype != torch.float32 and out.dtype != w.dtype:
             raise KernelError("grouped_linear: out is float32 or of the weights' type")
+        g_stride = 0
+        if gate is not None:
+            _want(gate, "gate", torch.float32, 2)
+            g_stride = gate.shape[1]
+            if gate.shape[0] < T or gate_offset + groups * n > g_stride:
+                raise KernelError("grouped_linear: the gate columns exceed the gate's row")
         listed = None
         if singles is not None:
             T, listed = min(T, singles.decode_cap), singles.data
@@ -1102,13 +1124,15 @@ class CudaOps:
             code = self.lib.hs_grouped_linear_mma(_ptr(out), _ptr(a), _ptr(w_nk), T, a.shape[1],
                                                   int(a_offset), gs, groups, n, k,
                                                   _DT[out.dtype], 3 if exact else 1,
-                                                  _ptr(listed), self._stream())
+                                                  _ptr(listed), _ptr(gate), g_stride,
+                                                  int(gate_offset), self._stream())
             if code != -1:
                 _check(code, f"grouped_linear_mma(groups={groups},n={n},k={k})")
                 return
         _check(self.lib.hs_grouped_linear(_ptr(out), _ptr(a), _ptr(w), T, a.shape[1],
                                           int(a_offset), gs, groups, n, k, _DT[w.dtype],
-                                          _DT[out.dtype], _ptr(listed), int(parts), self._stream()),
+                                          _DT[out.dtype], _ptr(listed), int(parts), _ptr(gate),
+                                          g_stride, int(gate_offset), self._stream()),
                f"grouped_linear(groups={groups},n={n},k={k})")
 
     # -- attention over a shared latent ---------------------------------------------------
@@ -1245,15 +1269,17 @@ class CudaOps:
     def latent_prompt_rows(self, plan, n_requests, *, n_heads, dim, rot_dim, vdim, rank, window,
                            scale) -> int:
         """Rows of the dense blocks with which the plan's prompt portions run in expanded form
-        (each portion's tokens and the window - 1 positions before them), or 0 when the kernels
-        do not take the sizes or the step has no portion."""
-        if (plan is None or plan.tile_cap <= 0 or window <= 0 or not self.tensor_cores
+        (each portion's tokens and the window - 1 positions before them; without a window all
+        positions before them), or 0 when the kernels do not take the sizes or the step has no
+        portion."""
+        if (plan is None or plan.tile_cap <= 0 or window < 0 or not self.tensor_cores
                 or not self.latent_expanded):
             return 0
         if not self.lib.hs_latent_prefill_tc_takes(int(dim), int(rot_dim), int(vdim), int(rank),
                                                    int(window), float(scale)):
             return 0
-        rows = plan.n_rows + min(n_requests, plan.tile_cap) * (window - 1)
+        rows = plan.n_rows + min(n_requests, plan.tile_cap) * (window - 1) if window \
+            else plan.prompt_rows
         return rows if 2 * rows * n_heads * (dim + vdim) <= self.LATENT_EXPANDED_BYTES else 0
 
     def latent_gather(self, lat, rope, q_out, base, q, pool, table, req_start, req_len, tok_pos,
@@ -1274,7 +1300,7 @@ class CudaOps:
         pad = -(-dim // 64) * 64
         if lat.shape[1] != rank or tuple(rope.shape) != (lat.shape[0], 64) or rot_dim > 64 or \
                 q_out.shape[1] != n_heads * (pad + 64) or q.shape[0] < T or \
-                q.shape[1] != n_heads * (dim + rot_dim) or pool.numel() % (page_size * W):
+                q.shape[1] < n_heads * (dim + rot_dim) or pool.numel() % (page_size * W):
             raise KernelError("latent_gather: shapes do not fit")
         if table.shape[0] < R or req_start.shape[0] < R or req_len.shape[0] < R or \
                 tok_pos.shape[0] < T or tok_req.shape[0] < T:
@@ -1283,14 +1309,15 @@ class CudaOps:
         _check(self.lib.hs_latent_gather(
             _ptr(lat), _ptr(rope), _ptr(q_out), _ptr(base), _ptr(q), _ptr(pool), _ptr(table),
             _ptr(req_start), _ptr(req_len), _ptr(tok_pos), _ptr(tok_req), R, T, lat.shape[0],
-            int(window), DECODE_MAX_NEW, rank, rot_dim, n_heads, dim, page_size,
+            int(window), DECODE_MAX_NEW, rank, rot_dim, n_heads, dim, q.shape[1], page_size,
             pool.numel() // (page_size * W), table.shape[1], _ptr(freq),
             int(rot_dims) if freq is not None else 0, _ptr(status), self._stream()),
             f"latent_gather(rank={rank},dim={dim})")
 
     def latent_prompt_attention(self, out, q, kv, rope, base, plan, *, n_heads, dim, rot_dim, vdim,
-                                rank, window, scale, status):
-        """Softmax attention of the plan's prompt portions over the last ``window`` positions:
+                                rank, window, scale, status, gate=None, gate_offset=0):
+        """Softmax attention of the plan's prompt portions over the last ``window`` positions (0:
+        over all), with ``gate`` (float32 [T, *]) times sigmoid(gate[t, gate_offset + column]):
         ``q`` as ``latent_gather`` left it, ``kv`` [rows, n_heads * (dim + vdim)] the expanded
         keys of all heads, then the values; ``out`` [T, n_heads * vdim] bfloat16 (rows of single-
         query tokens are left alone)."""
@@ -1302,12 +1329,18 @@ class CudaOps:
         if out.shape[1] != n_heads * vdim or tuple(q.shape) != (T, n_heads * (pad + 64)) or \
                 kv.shape[1] != n_heads * (dim + vdim) or tuple(rope.shape) != (rows, 64):
             raise KernelError("latent_prompt_attention: shapes do not fit")
+        g_stride = 0
+        if gate is not None:
+            _want(gate, "gate", torch.float32, 2)
+            g_stride = gate.shape[1]
+            if gate.shape[0] < T or gate_offset + n_heads * vdim > g_stride:
+                raise KernelError("latent_prompt_attention: the gate columns exceed the gate's row")
         self.launches += 1
         _check(self.lib.hs_latent_prefill_tc(
             _ptr(out), _ptr(q), _ptr(kv), _ptr(rope), _ptr(base), _ptr(plan.data),
             4 + plan_decode_ints(plan.n_rows), plan.tile_cap, T, rows, n_heads, dim, rot_dim, vdim,
-            rank, int(window), float(scale), _ptr(status), self._stream()),
-            f"latent_prompt_attention(dim={dim},rot_dim={rot_dim},vdim={vdim})")
+            rank, int(window), float(scale), _ptr(gate), g_stride, int(gate_offset), _ptr(status),
+            self._stream()), f"latent_prompt_attention(dim={dim},rot_dim={rot_dim},vdim={vdim})")
 
     # -- the gated delta rule ---------------------------------------------------------------
     @staticmethod
@@ -2075,10 +2108,12 @@ class CudaOps:
             self._stream()), f"timemix_recurrence(dim={dim})")
 
     def head_norm_gate(self, out, o, weight, gate, *, gate_offset, heads, dim, eps,
-                       gate_act="silu", out_scale=1.0):
+                       gate_act="silu", out_scale=1.0, gate_first=False):
         """out[t, h] = o[t, h] / rms(o[t, h]) (* weight) * act(gate columns) * out_scale for
         every head h of ``dim`` numbers; ``gate`` is float32 [T, *] with the head's columns from
-        ``gate_offset`` on, ``gate_act`` silu or sigmoid; weight and gate may be None."""
+        ``gate_offset`` on, ``gate_act`` silu or sigmoid; weight and gate may be None.  With
+        ``gate_first`` o is multiplied by the activated gate before its root mean square is
+        taken."""
         _want(out, "out", _FLOATS, 2)
         _want(o, "o", torch.float32, 2)
         T = out.shape[0]
@@ -2094,13 +2129,15 @@ class CudaOps:
             g_stride = gate.shape[1]
             if gate.shape[0] < T or gate_offset + heads * dim > g_stride:
                 raise KernelError("head_norm_gate: the gate columns exceed the gate's row")
+        if gate_first and gate is None:
+            raise KernelError("head_norm_gate: no gate to apply first")
         if gate_act not in ("silu", "sigmoid"):
             raise KernelError(f"head_norm_gate: gate activation {gate_act!r} not taken")
         self.launches += 1
         _check(self.lib.hs_head_norm_gate(
             _ptr(out), _ptr(o), _ptr(weight), _ptr(gate), g_stride, int(gate_offset), T, heads,
-            dim, float(eps), int(gate_act == "silu"), float(out_scale), _DT[out.dtype],
-            self._stream()), f"head_norm_gate(dim={dim})")
+            dim, float(eps), int(gate_act == "silu"), float(out_scale), int(bool(gate_first)),
+            _DT[out.dtype], self._stream()), f"head_norm_gate(dim={dim})")
 
     def gather_mul(self, out, g, table, tok_ids, tok_req, *, col_offset, feedback=None):
         """out[t, c] = g[t, c] * table[token[t], col_offset + c] (``g`` float32, ``out`` and
@@ -2144,10 +2181,13 @@ class CudaOps:
     # -- attention with a distance slope, a window and kept first tokens ---------------------
     def span_prepare(self, q_out, pool, proj, table, tok_pos, tok_req, *, n_heads, n_kv_heads,
                      head_dim, value_dim, q_off, k_off, v_off, qk_norm, eps, writes, page_size,
-                     status):
+                     status, wq=None, wk=None, freq=None, rot_dims=0):
         """From float32 projection rows: q (columns from ``q_off``) to ``q_out`` (float32), and
         with ``writes`` the row [k | v] of every key/value head into the token's page; with
-        ``qk_norm`` q and k are divided by their root mean square per head first.  ``v_off``
+        ``qk_norm`` q and k are divided by their root mean square per head first, with ``wq`` and
+        ``wk`` (one weight per number) each over its whole projection and weighted; with ``freq``
+        they are then turned on each head's first ``rot_dims`` numbers (number i pairs with
+        i + rot_dims / 2).  ``v_off``
         None: the values are the keys as projected (before the norm).  ``pool`` is
         [pages, kv_heads, page_size, head_dim + value_dim]."""
         _want(q_out, "q_out", torch.float32, 2)
@@ -2159,21 +2199,30 @@ class CudaOps:
             raise KernelError("span_prepare: the rows do not fit the heads")
         if writes and k_off is None:
             raise KernelError("span_prepare: a layer that writes its rows has key columns")
+        for w, n, nm in ((wq, H * D, "wq"), (wk, G * D, "wk")):
+            if w is not None and _want(w, nm, torch.float32, 1).shape[0] != n:
+                raise KernelError(f"span_prepare: {nm} has one weight per number")
+        if freq is None:
+            rot_dims = 0
+        elif _want(freq, "freq", torch.float32, 1).shape[0] < rot_dims // 2:
+            raise KernelError("span_prepare: one frequency per turned pair")
         self.launches += 1
         _check(self.lib.hs_span_prepare(
             _ptr(q_out), _ptr(pool), _ptr(proj), proj.shape[1], int(q_off),
             -1 if k_off is None else int(k_off), -1 if v_off is None else int(v_off), _ptr(table),
             table.shape[1], pool.numel() // (G * page_size * (D + V)), _ptr(tok_pos),
             _ptr(tok_req), q_out.shape[0], H, G, D, V, int(bool(qk_norm)), float(eps),
-            int(page_size), int(bool(writes)), _DT[pool.dtype], _ptr(status), self._stream()),
+            int(page_size), int(bool(writes)), _ptr(wq), _ptr(wk), _ptr(freq), int(rot_dims),
+            _DT[pool.dtype], _ptr(status), self._stream()),
             f"span_prepare(head_dim={D},value_dim={V})")
 
     def span_attention(self, out, q, pool, table, tok_pos, tok_req, *, n_heads, n_kv_heads,
                        head_dim, value_dim, scale, slopes, window, keep_first, gate, gate_offset,
-                       out_scale, page_size, status, plan=None):
+                       out_scale, page_size, status, plan=None, softcap=0.0, sinks=None):
         """Per token at position i and query head h: softmax over the keys j <= i with
         i - j < window (0: all) or j < keep_first of (q . k) * scale - slopes[h] * (i - j)
-        (``slopes`` float32 [heads] or None); the head's output times sigmoid(gate[t,
+        (``slopes`` float32 [heads] or None), with ``softcap`` c bent to c * tanh(score / c);
+        with ``sinks`` (float32 [heads]) the denominator also holds exp(sinks[h]); the head's output times sigmoid(gate[t,
         gate_offset + h * value_dim + e]) (``gate`` float32 [T, *] or None) times
         ``out_scale``.  With the step's ``plan`` and a bfloat16 cache the plan's tiles (prompt
         portions) run on the tensor cores and its single-query tokens on the CUDA cores;
@@ -2191,6 +2240,10 @@ class CudaOps:
             _want(slopes, "slopes", torch.float32, 1)
             if slopes.shape[0] != H:
                 raise KernelError("span_attention: one slope per head")
+        if sinks is not None and _want(sinks, "sinks", torch.float32, 1).shape[0] != H:
+            raise KernelError("span_attention: one sink per head")
+        if softcap < 0:
+            raise KernelError("span_attention: a cap is positive (0: none)")
         g_stride = 0
         if gate is not None:
             _want(gate, "gate", torch.float32, 2)
@@ -2208,7 +2261,8 @@ class CudaOps:
                 _ptr(d[4 + plan_decode_ints(plan.n_rows):]), _ptr(d), plan.tile_cap,
                 _ptr(self._scratch_buffer("span_counter", 1, torch.int32)), _ptr(slopes),
                 _ptr(gate), g_stride, int(gate_offset), float(out_scale), H, G, D, V, int(window),
-                int(keep_first), float(scale), int(page_size), _ptr(status), self._stream())
+                int(keep_first), float(scale), int(page_size), float(softcap), _ptr(sinks),
+                _ptr(status), self._stream())
             if code != -1:
                 _check(code, f"span_attention_prefill(head_dim={D},value_dim={V})")
                 self.launches += 1
@@ -2221,8 +2275,132 @@ class CudaOps:
             _ptr(out), _ptr(q), _ptr(pool), _ptr(table), table.shape[1], num_pages, _ptr(tok_pos),
             _ptr(tok_req), _ptr(slopes), _ptr(gate), g_stride, int(gate_offset), float(out_scale),
             T, H, G, D, V, int(window), int(keep_first), float(scale), int(page_size),
-            _DT[pool.dtype], _DT[out.dtype], _ptr(listed), _ptr(head), _ptr(status),
-            self._stream()), f"span_attention(head_dim={D},value_dim={V})")
+            _DT[pool.dtype], _DT[out.dtype], _ptr(listed), _ptr(head), float(softcap), _ptr(sinks),
+            _ptr(status), self._stream()), f"span_attention(head_dim={D},value_dim={V})")
+
+    # -- several copies of the stream --------------------------------------------------------
+    def hyper_mix(self, dst, src, y=None, *, streams, mix=None, write=None, read=None, u=None,
+                  out=None, norm=None):
+        """Behind a sublayer with output ``y`` (float32 [T, width]): copy t of a token's stream
+        becomes sum_s mix[s, t] * copy s + write[t] * y, all from the old ones; ``src`` and
+        ``dst`` are float32 [T, streams * width] and may be the same (``src`` may be [T, width]:
+        one row that stands for all copies; ``dst`` None: the copies are not kept).  Without
+        ``y`` the copies stay as they are.  ``u`` (float32 [T, width]) receives sum_t read[t] *
+        copy t of the new ones (``read`` None: their plain sum), and with ``norm = (weight, eps)``
+        ``out`` its root-mean-square norm times the weight."""
+        _want(src, "src", torch.float32, 2)
+        like = next((v for v in (out, u, y) if v is not None), None)
+        if like is None:
+            raise KernelError("hyper_mix: nothing to form")
+        n, W = src.shape[0], like.shape[1]
+        rows = src.shape[1] // W
+        if src.shape[1] != rows * W or rows not in (1, streams):
+            raise KernelError("hyper_mix: src is [T, streams * width] or [T, width]")
+        if y is not None:
+            _want(y, "y", torch.float32, 2)
+            _want(mix, "mix", torch.float32, 2)
+            _want(write, "write", torch.float32, 1)
+            if y.shape[0] < n or y.shape[1] != W or tuple(mix.shape) != (streams, streams) \
+                    or write.shape[0] != streams:
+                raise KernelError("hyper_mix: the sublayer's output does not fit")
+        if dst is not None and tuple(_want(dst, "dst", torch.float32, 2).shape) != (n, streams * W):
+            raise KernelError("hyper_mix: dst is [T, streams * width]")
+        if read is not None and _want(read, "read", torch.float32, 1).shape[0] != streams:
+            raise KernelError("hyper_mix: one number per copy")
+        if u is not None and tuple(_want(u, "u", torch.float32, 2).shape) != (n, W):
+            raise KernelError("hyper_mix: u is [T, width]")
+        if (out is None) != (norm is None):
+            raise KernelError("hyper_mix: out and norm come together")
+        weight, eps = norm if norm is not None else (None, 0.0)
+        if out is not None:
+            _want(out, "out", _FLOATS, 2)
+            _want(weight, "weight", torch.float32, 1)
+            if tuple(out.shape) != (n, W) or weight.shape[0] != W:
+                raise KernelError("hyper_mix: out / weight do not fit")
+        self.launches += 1
+        _check(self.lib.hs_hyper_mix(
+            _ptr(dst), _ptr(src), rows, _ptr(y), int(streams), _ptr(mix), _ptr(write), _ptr(read), n,
+            W, _ptr(u), _ptr(out), _ptr(weight), float(eps), _DT[out.dtype] if out is not None else 0,
+            self._stream()), f"hyper_mix(streams={streams},width={W})")
+
+    # -- the state-space recurrence -----------------------------------------------------------
+    def ssm_rows_dtype(self, dtype, n_tokens, sizes):
+        """The type in which ``ssm_prepare`` is to leave the activated rows of such a step."""
+        return torch.float32
+
+    @staticmethod
+    def _ssm_sizes(proj, state, x_off, heads, groups, state_dim, vdim, taps):
+        C = heads * vdim + 2 * groups * state_dim
+        _want(proj, "proj", torch.float32, 2)
+        _want(state, "state", torch.float32, 2)
+        if heads % groups or x_off + C + heads > proj.shape[1] \
+                or state.shape[1] < heads * state_dim * vdim + taps * C:
+            raise KernelError("state space: the projection's row or the state does not fit the sizes")
+        return C, (heads, groups, state_dim, vdim, taps, proj.shape[1], int(x_off), state.shape[1])
+
+    @staticmethod
+    def _ssm_conv(C, H, taps, conv_w, conv_b, dt_bias, a_log):
+        for t, nm, shape in ((conv_w, "conv_w", (taps, C)), (conv_b, "conv_b", (C,)),
+                             (dt_bias, "dt_bias", (H,)), (a_log, "a_log", (H,))):
+            if tuple(_want(t, nm, torch.float32).shape) != shape:
+                raise KernelError(f"state space: {nm} is {shape}")
+
+    def ssm_prepare(self, rows, step, proj, state, tok_req, tok_pos, req_start, req_slot, *,
+                    conv_w, conv_b, dt_bias, a_log, x_off, heads, groups, state_dim, vdim, taps):
+        """rows[t] = silu(conv(x | B | C columns of ``proj`` from ``x_off`` on)) (a causal
+        convolution per channel, ``conv_w`` [taps, channels], earlier inputs from the request's
+        slot of ``state``); step[t] = [dt | -exp(a_log) dt] with dt = softplus(the columns behind
+        them + dt_bias), one number per head each."""
+        C, sizes = self._ssm_sizes(proj, state, x_off, heads, groups, state_dim, vdim, taps)
+        self._ssm_conv(C, heads, taps, conv_w, conv_b, dt_bias, a_log)
+        _want(rows, "rows", _FLOATS, 2)
+        _want(step, "step", torch.float32, 2)
+        T = rows.shape[0]
+        if rows.shape[1] != C or tuple(step.shape) != (T, 2 * heads) or proj.shape[0] < T:
+            raise KernelError("ssm_prepare: rows / step do not fit")
+        self.launches += 1
+        _check(self.lib.hs_ssm_prepare(
+            _ptr(rows), _ptr(step), _ptr(proj), _ptr(state), _ptr(tok_req), _ptr(tok_pos),
+            _ptr(req_start), _ptr(req_slot), _ptr(conv_w), _ptr(conv_b), _ptr(dt_bias), _ptr(a_log),
+            T, *sizes, _DT[rows.dtype], self._stream()), f"ssm_prepare(channels={C})")
+
+    def ssm_recurrence(self, y, state, rows, step, proj, skip, tok_pos, req_start, req_len,
+                       req_slot, *, x_off, heads, groups, state_dim, vdim, taps):
+        """Per request and head, token after token on the float32 state S [state_dim, vdim] of the
+        request's slot: S <- exp(la) S + dt B x^T; y = S^T C + skip x, with rows and step as
+        ``ssm_prepare`` left them; the portion's last inputs (columns of ``proj``) go to the slot
+        for the tokens to come.  ``y`` is float32 [T, heads * vdim]."""
+        C, sizes = self._ssm_sizes(proj, state, x_off, heads, groups, state_dim, vdim, taps)
+        _want(y, "y", torch.float32, 2)
+        _want(rows, "rows", torch.float32, 2)
+        _want(step, "step", torch.float32, 2)
+        _want(skip, "skip", torch.float32, 1)
+        T = y.shape[0]
+        if y.shape[1] != heads * vdim or rows.shape[1] != C or rows.shape[0] < T \
+                or step.shape[0] < T or step.shape[1] != 2 * heads or skip.shape[0] != heads:
+            raise KernelError("ssm_recurrence: shapes do not fit")
+        self.launches += 1
+        _check(self.lib.hs_ssm_recurrence(
+            _ptr(y), _ptr(state), _ptr(rows), _ptr(step), _ptr(proj), _ptr(skip), _ptr(tok_pos),
+            _ptr(req_start), _ptr(req_len), _ptr(req_slot), req_start.shape[0], *sizes,
+            self._stream()), f"ssm_recurrence(state_dim={state_dim},vdim={vdim})")
+
+    def ssm_step(self, y, state, proj, skip, tok_req, tok_pos, req_slot, *, conv_w, conv_b,
+                 dt_bias, a_log, x_off, heads, groups, state_dim, vdim, taps):
+        """``ssm_prepare`` and ``ssm_recurrence`` in one launch, for a step in which every request
+        brings one token."""
+        C, sizes = self._ssm_sizes(proj, state, x_off, heads, groups, state_dim, vdim, taps)
+        self._ssm_conv(C, heads, taps, conv_w, conv_b, dt_bias, a_log)
+        _want(y, "y", torch.float32, 2)
+        _want(skip, "skip", torch.float32, 1)
+        T = y.shape[0]
+        if y.shape[1] != heads * vdim or proj.shape[0] < T or skip.shape[0] != heads:
+            raise KernelError("ssm_step: shapes do not fit")
+        self.launches += 1
+        _check(self.lib.hs_ssm_step(
+            _ptr(y), _ptr(state), _ptr(proj), _ptr(skip), _ptr(tok_req), _ptr(tok_pos),
+            _ptr(req_slot), _ptr(conv_w), _ptr(conv_b), _ptr(dt_bias), _ptr(a_log), T, *sizes,
+            self._stream()), f"ssm_step(state_dim={state_dim},vdim={vdim})")
 
     # -- sampling ---------------------------------------------------------------
     def argmax(self, out, logits):

@@ -76,6 +76,9 @@ class Part:
     # False for a part whose forward cannot be captured in a CUDA graph (its launches depend
     # on values read back to the host); a model with such a part is run without graphs.
     capturable: bool = True
+    # True for a part that sizes buffers by ``plan.prompt_rows``, which the runner then counts
+    # (and captures a graph per class of it).
+    counts_prompt_rows: bool = False
 
     def tensor_requests(self) -> dict[str, TensorRequest]:
         return {}

@@ -67,6 +67,8 @@ class LatentAttention(Mixer):
                           uv=value_up, sink=sink, o=out_weight, dq=q_down, dq_norm=q_down_norm,
                           g=gate)
         self.rot_pairing = rot_pairing
+        # without a window, prompts in expanded form need a row for every position they see
+        self.counts_prompt_rows = self.window == 0 and sink is None
         self.shares_cache = bool(shares_cache)
         self.q_width = self.H * (self.D + self.P)
         # columns of the input projection: the queries or their latent, then the key/value latent

@@ -388,6 +388,7 @@ class Model:
         self.schedule: tuple[LayerCall, ...] = spec.resolved_schedule()
         self.keeps_embedding = any(call.adds_embedding for call in self.schedule)
         self.capturable = all(part.capturable for part in self.parts())
+        self.counts_prompt_rows = any(part.counts_prompt_rows for part in self.parts())
         self._derive_cache()
         self.dtype = None
         self.device = None
