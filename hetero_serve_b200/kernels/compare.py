@@ -64,7 +64,7 @@ class TimedOps:
 
 _UNTIMED = {"stream", "register_kernel", "load_extension", "attention_plan_ints",
             "plan_attention", "make_plan", "decode_wide", "decode_splits",
-            "latent_prompt_rows"}
+            "latent_prompt_rows", "plan_prompt_rows", "ssm_rows_dtype"}
 
 
 def _contexts(batch):
@@ -261,6 +261,24 @@ def _flops_and_bytes(name, args, kw, batch):
                 last = start + n - 1
                 rows += last + 1 - max(0, start - win + 1) + max(0, (last - win + 1) // blk)
             return 2 * H * (D + V) * seen, _nbytes(out, q) + rows * G * (D + V) * pool.element_size()
+        if name == "hyper_mix":
+            dst, src = args[:2]
+            y = args[2] if len(args) > 2 else None
+            return 0, _nbytes(dst, src, y, kw.get("u"), kw.get("out"))
+        if name == "ssm_prepare":
+            rows, step = args[:2]
+            return 0, _nbytes(rows, step) + (rows.numel() + step.numel() // 2) * 4
+        if name == "ssm_recurrence":
+            y, _state, rows, step = args[:4]
+            H, N, V = kw["heads"], kw["state_dim"], kw["vdim"]
+            live = len([1 for _s, n in batch if n > 0])
+            return 5 * y.shape[0] * H * N * V, _nbytes(y, rows, step) + 2 * live * H * N * V * 4
+        if name == "ssm_step":
+            y = args[0]
+            H, G, N, V = kw["heads"], kw["groups"], kw["state_dim"], kw["vdim"]
+            C, live = H * V + 2 * G * N, len([1 for _s, n in batch if n > 0])
+            return (5 * y.shape[0] * H * N * V,
+                    _nbytes(y) + live * (2 * H * N * V + (kw["taps"] + 1) * C + H) * 4)
         if name in ("embed", "scale_", "rotary_pairs", "sample", "argmax", "kv_append"):
             return 0, _nbytes(args[0])
     except Exception:                                   # an estimate must never stop a step

@@ -168,3 +168,20 @@ def pivinex_case(request, pivinex_cases):
 def pivinex_planted(tmp_path_factory):
     import pivinex_cases as pc
     return {which: pc.planted_case(tmp_path_factory, which) for which in pc.PLANTED}
+
+
+@pytest.fixture(scope="session")
+def nukodra_cases(tmp_path_factory):
+    import nukodra_cases as nc
+    return nc.make_cases(tmp_path_factory)
+
+
+@pytest.fixture(params=["case_a", "case_b", "case_d"])
+def nukodra_case(request, nukodra_cases):
+    return nukodra_cases[request.param]
+
+
+@pytest.fixture(scope="session")
+def nukodra_planted(tmp_path_factory):
+    import nukodra_cases as nc
+    return {which: nc.planted_case(tmp_path_factory, which) for which in nc.PLANTED}
