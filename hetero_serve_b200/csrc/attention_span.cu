@@ -129,6 +129,111 @@ span_prepare_kernel(float* __restrict__ q_out, TC* __restrict__ pool,
   }
 }
 
+// The same for norms over the whole projections (or none), four numbers a thread: sizes, offsets and
+// half the turned extent in whole 16-byte pieces.
+template <typename TC>
+__global__ void __launch_bounds__(SA_WARPS * 32)
+span_prepare_wide_kernel(float* __restrict__ q_out, TC* __restrict__ pool,
+                         const float* __restrict__ proj, int proj_stride, int q_off, int k_off,
+                         int v_off, const int* __restrict__ table, int max_pages, int num_pages,
+                         const int* __restrict__ tok_pos, const int* __restrict__ tok_req, int H,
+                         int G, int D, int V, float eps, int page_size, int writes,
+                         const float* __restrict__ wq, const float* __restrict__ wk,
+                         const float* __restrict__ freq, int rot_dims, int* __restrict__ status) {
+  extern __shared__ __align__(16) float s_wide[];  // q [H*D] | k [G*D] | cosines, sines [rot_dims]
+  __shared__ float s_sq[2][SA_WARPS];
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const int r = tok_req[t];
+  if (r < 0) return;
+  const int pos = tok_pos[t], half = rot_dims >> 1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nq = H * D, nk = writes ? G * D : 0;
+  float* s_cos = s_wide + nq + nk;
+  float* s_sin = s_cos + half;
+  for (int i = threadIdx.x; i < half; i += SA_WARPS * 32) pair_angle(pos, freq[i], &s_cos[i], &s_sin[i]);
+  TC* row = nullptr;
+  if (writes) {
+    const int pi = pos / page_size;
+    const int page = (pos >= 0 && pi < max_pages) ? table[(size_t)r * max_pages + pi] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (threadIdx.x == 0) atomicOr(status, HS_STATUS_BAD_PAGE);
+    } else {
+      row = pool + ((size_t)page * G * page_size + (pos % page_size)) * (size_t)(D + V);
+    }
+  }
+  pdl_wait();
+  const float* pr = proj + (size_t)t * proj_stride;
+  auto put = [&](TC* dst, float4 v) {
+    if constexpr (sizeof(TC) == 4) {
+      *(float4*)dst = v;
+    } else {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      *(uint2*)dst = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+    }
+  };
+  float sq = 0.f, sk = 0.f;
+  for (int e = 4 * threadIdx.x; e < nq + nk; e += 4 * SA_WARPS * 32) {
+    const float4 v = *(const float4*)(pr + (e < nq ? q_off + e : k_off + e - nq));
+    *(float4*)(s_wide + e) = v;
+    const float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+    if (e < nq) sq += ss;
+    else sk += ss;
+  }
+  if (row) {                                       // values go as they are
+    const float* src = pr + (v_off < 0 ? k_off : v_off);
+    for (int e = 4 * threadIdx.x; e < G * V; e += 4 * SA_WARPS * 32) {
+      const int g = e / V, c = e - g * V;
+      put(row + (size_t)g * page_size * (D + V) + D + c, *(const float4*)(src + e));
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) {
+    s_sq[0][warp] = sq;
+    s_sq[1][warp] = sk;
+  }
+  __syncthreads();
+  float rq = 1.0f, rk = 1.0f;
+  if (wq) {
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < SA_WARPS; ++w) {
+      sq += s_sq[0][w];
+      sk += s_sq[1][w];
+    }
+    rq = 1.0f / sqrtf(sq / (float)(H * D) + eps);
+    rk = 1.0f / sqrtf(sk / (float)(G * D) + eps);
+  }
+  for (int e = 4 * threadIdx.x; e < nq + nk; e += 4 * SA_WARPS * 32) {
+    const bool is_q = e < nq;
+    const int at = is_q ? e : e - nq, g = at / D, c = at - g * D;
+    if (!is_q && !row) break;
+    const float rn = is_q ? rq : rk;
+    const float* wt = is_q ? wq : wk;
+    auto normed = [&](int i) {                     // the piece at i numbers from this one
+      float4 v = *(const float4*)(s_wide + e + i);
+      v = make_float4(v.x * rn, v.y * rn, v.z * rn, v.w * rn);
+      if (wt) {
+        const float4 w = *(const float4*)(wt + at + i);
+        v = make_float4(v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w);
+      }
+      return v;
+    };
+    float4 v = normed(0);
+    if (c < rot_dims) {
+      const bool low = c < half;
+      const float4 o = normed(low ? half : -half);
+      const float4 cs = *(const float4*)(s_cos + (low ? c : c - half));
+      float4 sn = *(const float4*)(s_sin + (low ? c : c - half));
+      if (low) sn = make_float4(-sn.x, -sn.y, -sn.z, -sn.w);
+      v = make_float4(v.x * cs.x + o.x * sn.x, v.y * cs.y + o.y * sn.y, v.z * cs.z + o.z * sn.z,
+                      v.w * cs.w + o.w * sn.w);
+    }
+    if (is_q) *(float4*)(q_out + (size_t)t * nq + e) = v;
+    else put(row + (size_t)g * page_size * (D + V) + c, v);
+  }
+}
+
 __device__ __forceinline__ float sa_dot(const float* __restrict__ k, const float* q, int D,
                                         bool vec) {
   float s = 0.f;
@@ -322,6 +427,22 @@ HS_EXPORT int hs_span_prepare(float* q_out, void* pool, const float* proj, int p
   if (smem > 40 * 1024) return HS_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
   cudaError_t e;
+  const size_t wide = ((size_t)(H + (writes ? G : 0)) * D + rot_dims) * sizeof(float);
+  if (!qk_norm && D % 4 == 0 && V % 4 == 0 && rot_dims % 8 == 0 && q_off % 4 == 0 &&
+      (!writes || (k_off % 4 == 0 && (v_off < 0 || v_off % 4 == 0))) && proj_stride % 4 == 0 &&
+      wide <= 47 * 1024 &&
+      !(((uintptr_t)q_out | (uintptr_t)pool | (uintptr_t)proj | (uintptr_t)wq | (uintptr_t)wk) & 15)) {
+#define HS_SPW(TC)                                                                                 \
+  e = hs_launch(hs::span_prepare_wide_kernel<TC>, dim3(n_tokens), dim3(hs::SA_WARPS * 32), wide, st, \
+                hs_pdl_enabled(), q_out, (TC*)pool, proj, proj_stride, q_off, k_off, v_off, table, \
+                max_pages, num_pages, tok_pos, tok_req, H, G, D, V, eps, page_size, writes, wq, wk, \
+                freq, rot_dims, status)
+    if (cache_dtype == HS_DT_BF16) HS_SPW(__nv_bfloat16);
+    else if (cache_dtype == HS_DT_F32) HS_SPW(float);
+    else return HS_ERR_UNSUPPORTED;
+#undef HS_SPW
+    return e == cudaSuccess ? HS_OK : (int)e;
+  }
   if (cache_dtype == HS_DT_BF16)
     e = hs_launch(hs::span_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(hs::SA_WARPS * 32),
                   smem, st, hs_pdl_enabled(), q_out, (__nv_bfloat16*)pool, proj, proj_stride, q_off,

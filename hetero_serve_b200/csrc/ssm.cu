@@ -50,7 +50,7 @@ __device__ __forceinline__ float ssm_conv(const float* __restrict__ own, int str
   return ssm_silu(acc);
 }
 
-constexpr int SP_TOK = 8;        // tokens a block of ssm_prepare walks
+constexpr int SP_TOK = 2;        // tokens a block of ssm_prepare walks
 
 // VEC: four channels a thread (every row and offset in whole 16-byte pieces)
 template <bool VEC, typename TR>

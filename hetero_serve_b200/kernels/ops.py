@@ -247,6 +247,9 @@ def _declare(lib) -> None:
         "hs_hyper_mix": [P, P, I, P, I, P, P, P, I, I, P, P, P, F, I, P],
         "hs_ssm_prepare": [P] * 12 + [I] * 10 + [P],
         "hs_ssm_recurrence": [P] * 10 + [I] * 9 + [P],
+        "hs_ssm_chunk_takes": [I, I, I, I],
+        "hs_ssm_chunk_slots": [I, I],
+        "hs_ssm_chunked": [P] * 10 + [I] * 10 + [P, P, P],
         "hs_ssm_step": [P] * 11 + [I] * 9 + [P],
         "hs_embed_norm": [P, P, P, P, P, I, I, I, I, P, I, P, P, F, P, P, P, F, I, P, P],
         "hs_residual_mix": [P, P, P, P, P, P, I, I, P, P, P, F, I, P],
@@ -356,6 +359,8 @@ class CudaOps:
         self.latent_mma = True      # prompt portions of latent attention on the tensor cores
         self.biased_mma = True      # prompt portions of the biased chunk attention likewise
         self.pooled_mma = True      # ... and of the attention over a window and pooled blocks
+        self.ssm_chunk_rows = 64    # from this many tokens a step on
+        self.ssm_chunks = True      # prompt portions of a state-space recurrence as chunks likewise
         self.span_mma = True        # ... and of the attention with a distance slope and a window
         self.folds_pooled_means = True   # pooled_prepare takes the companion pool (single tokens)
         self.lightning_bulk_rows = 64   # from this many tokens a step on, lightning attention
@@ -2325,7 +2330,13 @@ class CudaOps:
 
     # -- the state-space recurrence -----------------------------------------------------------
     def ssm_rows_dtype(self, dtype, n_tokens, sizes):
-        """The type in which ``ssm_prepare`` is to leave the activated rows of such a step."""
+        """The type in which ``ssm_prepare`` is to leave the activated rows of such a step:
+        bfloat16 where ``ssm_recurrence`` then runs in chunks on the tensor cores."""
+        H, G, N, V = (sizes[k] for k in ("heads", "groups", "state_dim", "vdim"))
+        if (dtype == torch.bfloat16 and self.tensor_cores and self.ssm_chunks
+                and n_tokens >= self.ssm_chunk_rows and self.lib.hs_ssm_chunk_takes(H, G, N, V)
+                and (H * N * V + sizes["taps"] * (H * V + 2 * G * N)) % 4 == 0):
+            return torch.bfloat16
         return torch.float32
 
     @staticmethod
@@ -2366,19 +2377,31 @@ class CudaOps:
 
     def ssm_recurrence(self, y, state, rows, step, proj, skip, tok_pos, req_start, req_len,
                        req_slot, *, x_off, heads, groups, state_dim, vdim, taps):
-        """Per request and head, token after token on the float32 state S [state_dim, vdim] of the
-        request's slot: S <- exp(la) S + dt B x^T; y = S^T C + skip x, with rows and step as
+        """Per request and head, on the float32 state S [state_dim, vdim] of the request's slot,
+        token after token or (rows in bfloat16) in chunks on the tensor cores:
+        S <- exp(la) S + dt B x^T; y = S^T C + skip x, with rows and step as
         ``ssm_prepare`` left them; the portion's last inputs (columns of ``proj``) go to the slot
         for the tokens to come.  ``y`` is float32 [T, heads * vdim]."""
         C, sizes = self._ssm_sizes(proj, state, x_off, heads, groups, state_dim, vdim, taps)
         _want(y, "y", torch.float32, 2)
-        _want(rows, "rows", torch.float32, 2)
+        _want(rows, "rows", _FLOATS, 2)
         _want(step, "step", torch.float32, 2)
         _want(skip, "skip", torch.float32, 1)
         T = y.shape[0]
         if y.shape[1] != heads * vdim or rows.shape[1] != C or rows.shape[0] < T \
                 or step.shape[0] < T or step.shape[1] != 2 * heads or skip.shape[0] != heads:
             raise KernelError("ssm_recurrence: shapes do not fit")
+        if rows.dtype == torch.bfloat16:
+            R = req_start.shape[0]
+            slots = self.lib.hs_ssm_chunk_slots(T, R)
+            states = self._scratch_buffer("ssm_states", slots * heads * state_dim * vdim, torch.float32)
+            whole = self._scratch_buffer("ssm_decays", slots * heads, torch.float32)
+            self.launches += 3
+            _check(self.lib.hs_ssm_chunked(
+                _ptr(y), _ptr(state), _ptr(rows), _ptr(step), _ptr(proj), _ptr(skip), _ptr(tok_pos),
+                _ptr(req_start), _ptr(req_len), _ptr(req_slot), R, T, *sizes, _ptr(states), _ptr(whole),
+                self._stream()), f"ssm_chunked(state_dim={state_dim},vdim={vdim})")
+            return
         self.launches += 1
         _check(self.lib.hs_ssm_recurrence(
             _ptr(y), _ptr(state), _ptr(rows), _ptr(step), _ptr(proj), _ptr(skip), _ptr(tok_pos),
