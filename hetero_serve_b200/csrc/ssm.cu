@@ -126,7 +126,7 @@ __device__ __forceinline__ void ssm_keep_inputs(float* __restrict__ ring,
 constexpr int SR_THREADS = 128;
 constexpr int SR_ROWS = 16;          // state rows a thread keeps
 constexpr int SR_PART = SR_ROWS + 4; // floats between two parts' rows of a token: distinct banks
-constexpr int SR_TOK = 16;           // tokens staged at a time (8 when N is above 128)
+constexpr int SR_TOK = 16;           // tokens staged at a time (8 when N is above 128, 4 above 256)
 
 __device__ __forceinline__ void sr_cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(
@@ -436,13 +436,13 @@ HS_EXPORT int hs_ssm_recurrence(float* y, float* state, const float* rows, const
       !req_slot)
     return HS_ERR_ARGUMENT;
   SsmShape s;
-  if (!ssm_shape(s, H, G, N, V, taps, stride, x_off, state_stride) || N > 16 * SR_ROWS)
+  if (!ssm_shape(s, H, G, N, V, taps, stride, x_off, state_stride) || N > 32 * SR_ROWS)
     return HS_ERR_UNSUPPORTED;
   if (n_requests <= 0) return HS_OK;
   if (n_requests > 65535 || H > 65535) return HS_ERR_TOO_LARGE;
   int P = 1;
   while (P * SR_ROWS < N) P *= 2;
-  const int cols = SR_THREADS / P, ntok = P * SR_ROWS > 128 ? SR_TOK / 2 : SR_TOK;
+  const int cols = SR_THREADS / P, ntok = P <= 8 ? SR_TOK : P == 16 ? SR_TOK / 2 : SR_TOK / 4;
   const int vec = N % 4 == 0 && V % 4 == 0 && cols % 4 == 0 && !((uintptr_t)rows & 15) ? 1 : 0;
   const size_t smem = (size_t)2 * ntok * (2 * P * SR_PART + cols + 2) * sizeof(float);
   if (smem > 48 * 1024) return HS_ERR_UNSUPPORTED;

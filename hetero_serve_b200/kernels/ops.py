@@ -244,6 +244,8 @@ def _declare(lib) -> None:
                               I, P, P, F, P, P, P],
         "hs_span_attention_prefill": [P, P, P, P, I, I, P, P, I, P, P, P, I, I, F, I, I, I, I, I, I,
                                       F, I, F, P, P, P],
+        "hs_span_decode_mma": [P, P, P, P, I, I, P, I, P, P, I, I, F, I, I, I, I, I, I, F, I, F, P, P,
+                               P],
         "hs_hyper_mix": [P, P, I, P, I, P, P, P, I, I, P, P, P, F, I, P],
         "hs_ssm_prepare": [P] * 12 + [I] * 10 + [P],
         "hs_ssm_recurrence": [P] * 10 + [I] * 9 + [P],
@@ -361,6 +363,9 @@ class CudaOps:
         self.pooled_mma = True      # ... and of the attention over a window and pooled blocks
         self.ssm_chunk_rows = 64    # from this many tokens a step on
         self.ssm_chunks = True      # prompt portions of a state-space recurrence as chunks likewise
+        self.span_decode_mma = True     # single-query tokens of the latter likewise, where more than
+        self.span_decode_keys = 512     # so many keys may be visible (measured: 128 blocks on the
+        #                                 CUDA cores are through with 256 keys before the clusters)
         self.span_mma = True        # ... and of the attention with a distance slope and a window
         self.folds_pooled_means = True   # pooled_prepare takes the companion pool (single tokens)
         self.lightning_bulk_rows = 64   # from this many tokens a step on, lightning attention
@@ -2230,7 +2235,9 @@ class CudaOps:
         with ``sinks`` (float32 [heads]) the denominator also holds exp(sinks[h]); the head's output times sigmoid(gate[t,
         gate_offset + h * value_dim + e]) (``gate`` float32 [T, *] or None) times
         ``out_scale``.  With the step's ``plan`` and a bfloat16 cache the plan's tiles (prompt
-        portions) run on the tensor cores and its single-query tokens on the CUDA cores;
+        portions) run on the tensor cores, and so do its single-query tokens when many keys may be
+        visible, with queries and weights in several bfloat16 terms (float32's mantissa), a cluster
+        of blocks a token;
         without a plan, in float32 and for sizes the tile kernel does not take every token
         runs on the CUDA cores."""
         _want(out, "out", _FLOATS, 2)
@@ -2273,8 +2280,22 @@ class CudaOps:
                 self.launches += 1
                 if plan.decode_cap == 0:
                     return
-                listed, head = d[4:], d         # the CUDA-core kernel takes the single tokens
+                listed, head = d[4:], d         # what is left are the single tokens
                 T = plan.decode_cap
+        if (plan is not None and out.dtype == torch.bfloat16 and self.tensor_cores
+                and self.span_decode_mma and plan.decode_cap > 0
+                and not 0 < window + keep_first * (window > 0) <= self.span_decode_keys
+                and (listed is not None or plan.tile_cap == 0)):
+            code = self.lib.hs_span_decode_mma(
+                _ptr(out), _ptr(q), _ptr(pool), _ptr(table), table.shape[1], num_pages,
+                _ptr(plan.data), plan.decode_cap, _ptr(slopes), _ptr(gate), g_stride,
+                int(gate_offset), float(out_scale), H, G, D, V, int(window), int(keep_first),
+                float(scale), int(page_size), float(softcap), _ptr(sinks), _ptr(status),
+                self._stream())
+            if code != -1:
+                _check(code, f"span_decode_mma(head_dim={D},value_dim={V})")
+                self.launches += 1
+                return
         self.launches += 1
         _check(self.lib.hs_span_attention(
             _ptr(out), _ptr(q), _ptr(pool), _ptr(table), table.shape[1], num_pages, _ptr(tok_pos),

@@ -102,11 +102,15 @@ def _plain_attention(rows, H, G, D, V, offs, wq, wk, rot, scale, window, cap, si
     (6, 2, 48, 48, 70, 48, 0.0, True), (6, 2, 96, 96, 96, 96, 30.0, True),
     (20, 1, 64, 128, 33, 0, 10.0, True), (2, 1, 112, 80, 130, 112, 30.0, True),
     (16, 4, 72, 104, 64, 24, 12.0, True), (4, 2, 256, 64, 40, 128, 30.0, True)])
-@pytest.mark.parametrize("planned", [False, True])
-def test_span_attention(ops, dtype, tol, H, G, D, V, window, rot, cap, sinks, planned):
+@pytest.mark.parametrize("planned", ["no", "yes", "clusters"])
+def test_span_attention(ops, monkeypatch, dtype, tol, H, G, D, V, window, rot, cap, sinks, planned):
     """Two requests whose pages are scattered over the pool, in portions that end inside pages and
     windows; then single tokens.  Every position is compared.  The pages behind the window are
-    taken out of the table: nothing may look them up.  Unused rows of the pool are NaN."""
+    taken out of the table: nothing may look them up.  Unused rows of the pool are NaN.  With the
+    step's work lists portions run as tiles; "clusters": single tokens on the kernel for many keys,
+    whose products keep float32's mantissa, whatever the window."""
+    if planned == "clusters":
+        monkeypatch.setattr(ops, "span_decode_keys", 0)
     eps, page, scale = 1e-5, 16, 2.0 / math.sqrt(D)
     q_off = 8
     k_off = q_off + H * D
@@ -153,7 +157,7 @@ def test_span_attention(ops, dtype, tol, H, G, D, V, window, rot, cap, sinks, pl
                 tab[row, :max(0, fed[r] - window + 1) // page] = -1
         out = torch.full((T, H * V), float("nan"), dtype=dtype, device=DEV)
         work = ops.make_plan([(row, row, fed[r], k) for row, (r, k) in enumerate(step)], T, page) \
-            if planned else None
+            if planned != "no" else None
         ops.span_attention(out, q, pool, tab, tok_pos, tok_req, scale=scale, slopes=None,
                            window=window, keep_first=0, gate=proj, gate_offset=g_off, out_scale=1.0,
                            plan=work, softcap=cap, sinks=sk, **sizes)
@@ -309,7 +313,8 @@ def _walk(xbc, dt, w, skip, H, G, N, V, state=None):
 
 
 SSM_SIZES = [(6, 2, 14, 10, 3), (4, 4, 8, 8, 1), (1, 1, 1, 8, 2), (5, 1, 9, 7, 5), (8, 2, 64, 32, 4),
-             (3, 1, 128, 64, 4), (4, 2, 48, 32, 3), (2, 1, 200, 96, 4), (4, 1, 16, 128, 4), (2, 2, 256, 16, 2)]
+             (3, 1, 128, 64, 4), (4, 2, 48, 32, 3), (2, 1, 200, 96, 4), (4, 1, 16, 128, 4), (2, 2, 256, 16, 2),
+             (2, 1, 500, 12, 4)]
 
 
 @pytest.mark.parametrize("H, G, N, V, taps", SSM_SIZES)
