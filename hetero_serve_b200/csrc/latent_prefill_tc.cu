@@ -17,6 +17,10 @@
 // positions 0 .. s + n - 1 and its rows follow those of the portions before r.  Rows nobody wrote
 // hold zeros or an earlier step's numbers: finite, and always masked.
 //
+// The second and third step serve attention over keys and values of the cache itself as well
+// (span_gather brings [all keys | all values] of a position into one dense row): query heads that
+// share a key/value head, no turned part, capped scores, a sink in the denominator.
+//
 // A block works on up to 128 consecutive queries of one request x one head, 128 keys a tile:
 //   warp 0      TMA producer: the queries once; per tile the key chunks of 64 numbers (the head's
 //               columns of the expanded rows, then the shared turned part) into two stages, the
@@ -136,6 +140,73 @@ latent_gather_kernel(__nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict_
   }
 }
 
+// The same for a cache of keys and values: dense rows [G keys of D | G values of V], queries padded.
+__global__ void __launch_bounds__(256)
+span_gather_kernel(__nv_bfloat16* __restrict__ kv, __nv_bfloat16* __restrict__ q_out,
+                   int* __restrict__ base, const float* __restrict__ q,
+                   const __nv_bfloat16* __restrict__ pool, const int* __restrict__ table,
+                   const int* __restrict__ req_start, const int* __restrict__ req_len,
+                   const int* __restrict__ tok_pos, const int* __restrict__ tok_req, int n_requests,
+                   int cap_rows, int window, int max_single, int H, int G, int D, int V, int q_pad_d,
+                   int page_size, int num_pages, int max_pages, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int n_gather = n_requests * LP_GATHER_BLOCKS;
+  if ((int)blockIdx.x < n_gather) {
+    const int r = blockIdx.x / LP_GATHER_BLOCKS, part = blockIdx.x - r * LP_GATHER_BLOCKS;
+    const int n = req_len[r];
+    if (n <= max_single) {
+      if (part == 0 && threadIdx.x == 0) base[r] = -1;
+      return;
+    }
+    const int pos0 = tok_pos[req_start[r]];
+    int lo = 0, row0 = 0;
+    if (window > 0) {
+      int before = 0;
+      for (int i = 0; i < r; ++i) before += req_len[i] > max_single;
+      lo = max(0, pos0 + 1 - window);
+      row0 = req_start[r] + before * (window - 1);
+    } else {
+      for (int i = 0; i < r; ++i)
+        if (req_len[i] > max_single) row0 += tok_pos[req_start[i]] + req_len[i];
+    }
+    const int rows = pos0 + n - lo;
+    if (part == 0 && threadIdx.x == 0) base[r] = row0 - lo;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int W = D + V, wq = W / 8, pieces = G * wq;
+    for (int i = part * 8 + warp; i < rows; i += LP_GATHER_BLOCKS * 8) {
+      const int row = row0 + i, p = lo + i, pi = p / page_size;
+      if (row >= cap_rows) break;                         // the caller's block is too small
+      const int page = pi < max_pages ? table[(size_t)r * max_pages + pi] : -1;
+      if (page < 0 || page >= num_pages) {
+        if (lane == 0) atomicOr(status, HS_STATUS_BAD_PAGE);
+        continue;
+      }
+      const __nv_bfloat16* src =
+          pool + ((size_t)page * G * page_size + (p - pi * page_size)) * (size_t)W;
+      __nv_bfloat16* dst = kv + (size_t)row * G * W;
+      for (int c = lane; c < pieces; c += 32) {
+        const int g = c / wq, e = (c - g * wq) * 8;
+        *(uint4*)(dst + (e < D ? g * D + e : G * D + g * V + e - D)) =
+            *(const uint4*)(src + (size_t)g * page_size * W + e);
+      }
+    }
+    return;
+  }
+  const int t = blockIdx.x - n_gather;
+  const int r = tok_req[t];
+  if (r < 0 || req_len[r] <= max_single) return;
+  const float* src = q + (size_t)t * H * D;
+  __nv_bfloat16* dst = q_out + (size_t)t * H * q_pad_d;
+  for (int i = 4 * threadIdx.x; i < H * q_pad_d; i += 4 * 256) {
+    const int h = i / q_pad_d, e = i - h * q_pad_d;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (e < D) v = *(const float4*)(src + (size_t)h * D + e);       // D is a multiple of 8
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *(uint2*)(dst + i) = make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
+  }
+}
+
 // ---- attend --------------------------------------------------------------------------------
 struct LatentTcParams {
   __nv_bfloat16* out;             // [tokens, heads * V]
@@ -143,7 +214,9 @@ struct LatentTcParams {
   const int* base;
   int* status;
   int tiles_off, n_heads, D, V, window, cap_rows;     // window: huge when there is none
-  float scale;
+  float scale, softcap;           // softcap 0: none
+  int kv_group, v_col;            // query heads of a key/value head; column of the first value
+  const float* sinks;             // [n_heads] or null
   const float* gate;              // [tokens, gate_stride] or null: column gate_off + h * V + e
   int gate_stride, gate_off;
 };
@@ -157,6 +230,10 @@ __device__ __forceinline__ float lp_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// cap * tanh(s / cap) = cap * (1 - 2 / (1 + e^(2 s / cap))), the exponent as z * in
+__device__ __forceinline__ float lp_cap(float z, float in, float cap) {
+  return cap * (1.0f - __fdividef(2.0f, 1.0f + lp_ex2(z * in)));
+}
 // values, N-contiguous, more than one 64-number chunk wide: the chunks lie 16 KB apart
 __device__ __forceinline__ uint64_t lp_value_desc(uint32_t saddr) {
   uint64_t d = make_smem_desc(saddr);
@@ -165,8 +242,8 @@ __device__ __forceinline__ uint64_t lp_value_desc(uint32_t saddr) {
   return d;
 }
 
-// NK: key chunks of 64 numbers (the turned part is the last); NV: value chunks
-template <int NK, int NV>
+// NK: key chunks of 64 numbers (with TURNED, the shared turned part is the last); NV: value chunks
+template <int NK, int NV, bool TURNED>
 __global__ void __launch_bounds__(LP_THREADS, 1)
 latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                          const __grid_constant__ CUtensorMap map_kv,
@@ -185,7 +262,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   if ((int)blockIdx.y >= p.plan[1]) return;
   const int4 ti = *(const int4*)(p.plan + p.tiles_off + 4 * blockIdx.y);
   const int tok0 = ti.x, nq = ti.y, r = ti.z, pos0 = ti.w;
-  const int h = blockIdx.x;
+  const int h = blockIdx.x, hk = h / p.kv_group;
   if (r < 0 || nq <= 0 || nq > LP_BQ || pos0 < 0) return;
   const int pos_last = pos0 + nq - 1;
   const int lo = max(0, pos0 + 1 - p.window);            // the oldest position a query here sees
@@ -228,9 +305,9 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         mbar_expect_tx(&bars[LB_K_FULL + st], NK * LP_CHUNK);
         uint8_t* dk = sK + st * NK * LP_CHUNK;
 #pragma unroll
-        for (int c = 0; c < NK - 1; ++c)
-          tma_load_2d(dk + c * LP_CHUNK, &map_kv, &bars[LB_K_FULL + st], h * p.D + c * 64, y);
-        tma_load_2d(dk + (NK - 1) * LP_CHUNK, &map_rope, &bars[LB_K_FULL + st], 0, y);
+        for (int c = 0; c < (TURNED ? NK - 1 : NK); ++c)
+          tma_load_2d(dk + c * LP_CHUNK, &map_kv, &bars[LB_K_FULL + st], hk * p.D + c * 64, y);
+        if (TURNED) tma_load_2d(dk + (NK - 1) * LP_CHUNK, &map_rope, &bars[LB_K_FULL + st], 0, y);
         return true;
       };
       mbar_expect_tx(&bars[LB_Q], NK * LP_CHUNK);
@@ -248,7 +325,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
         for (int c = 0; c < NV; ++c)
           tma_load_2d(sV + c * LP_CHUNK, &map_kv, &bars[LB_V_FULL],
-                      p.n_heads * p.D + h * p.V + c * 64, y);
+                      p.v_col + hk * p.V + c * 64, y);
       }
     }
   } else if (warp == 1) {
@@ -300,7 +377,11 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     const int row = qtr * 32 + lane;
     const int pos_r = min(pos0 + row, pos_last);           // rows past nq: finite, never stored
     const uint32_t lane_addr = tmem_base + ((uint32_t)(qtr * 32) << 16);
-    const float sl2 = p.scale * 1.4426950408889634f;
+    const bool capped = p.softcap > 0.f;
+    const float to2 = p.scale * 1.4426950408889634f;       // a score in units of log2(e)
+    const float sl2 = capped ? 1.0f : to2;                 // capped scores are in those units already
+    const float cap2 = p.softcap * 1.4426950408889634f;
+    const float cap_in = capped ? 2.0f * to2 / p.softcap : 0.f;      // 2 log2(e) scale / cap
     float m = -INFINITY, l = 0.f, corr_pending = 1.f;
     constexpr int OC = NV * 32;                            // output columns of this thread
     float o[OC];
@@ -339,6 +420,13 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       tmem_ld32(s_addr, va);
       tmem_ld32(s_addr + 32, vb);
       tmem_ld_wait();
+      if (capped) {                                        // cap * tanh(s / cap)
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          va[j] = __float_as_uint(lp_cap(__uint_as_float(va[j]), cap_in, cap2));
+          vb[j] = __float_as_uint(lp_cap(__uint_as_float(vb[j]), cap_in, cap2));
+        }
+      }
       if (edge) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
@@ -399,9 +487,14 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     if (ok) ok = accumulate_o(n_kv - 1);
     s_l[half][row] = l;
     asm volatile("bar.sync %0, 64;" ::"r"(1 + qtr) : "memory");
-    const float l_all = l + s_l[half ^ 1][row];
+    float l_all = l + s_l[half ^ 1][row], keep = 1.f;
+    if (p.sinks) {
+      const float sk = p.sinks[h] * 1.4426950408889634f, top = fmaxf(m, sk);
+      keep = lp_ex2(m - top);
+      l_all = l_all * keep + lp_ex2(sk - top);
+    }
     if (ok && row < nq) {
-      const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+      const float inv = l_all > 0.f ? keep / l_all : 0.f;
       __nv_bfloat16* orow = p.out + ((size_t)(tok0 + row) * p.n_heads + h) * p.V;
       const float* grow = p.gate ? p.gate + (size_t)(tok0 + row) * p.gate_stride + p.gate_off +
                                        (size_t)h * p.V + half * OC
@@ -500,35 +593,73 @@ HS_EXPORT int hs_latent_gather(void* lat, void* rope, void* q_out, int* base, co
   return e == cudaSuccess ? HS_OK : (int)e;
 }
 
-// kv [cap_rows, n_heads * (D + V)]: the expanded keys of all heads, then the values.
+// Whether prompt portions over a cache of keys and values take these sizes: keys of up to 192
+// numbers, values of up to 128, in whole 16-byte pieces.
+HS_EXPORT int hs_span_prefill_tc_takes(int H, int G, int D, int V, int window, float scale) {
+  return H > 0 && G > 0 && H % G == 0 && D > 0 && D <= 192 && D % 8 == 0 && V > 0 && V <= 128 &&
+                 V % 8 == 0 && window >= 0 && scale > 0.f
+             ? 1
+             : 0;
+}
+
+// kv [cap_rows, G * (D + V)], q_out [n_tokens, H * pad64(D)], base [n_requests]; q [n_tokens, H * D]
+// float32; pool [pages][G][page_size][D + V].
+HS_EXPORT int hs_span_gather(void* kv, void* q_out, int* base, const float* q, const void* pool,
+                             const int* table, const int* req_start, const int* req_len,
+                             const int* tok_pos, const int* tok_req, int n_requests, int n_tokens,
+                             int cap_rows, int window, int max_single, int H, int G, int D, int V,
+                             int page_size, int num_pages, int max_pages, int* status, void* stream) {
+  if (!kv || !q_out || !base || !q || !pool || !table || !req_start || !req_len || !tok_pos ||
+      !tok_req || !status)
+    return HS_ERR_ARGUMENT;
+  if (!hs_span_prefill_tc_takes(H, G, D, V, window, 1.f) || page_size <= 0 ||
+      (((uintptr_t)kv | (uintptr_t)q_out | (uintptr_t)q | (uintptr_t)pool) & 15))
+    return HS_ERR_UNSUPPORTED;
+  if (n_requests <= 0 || n_tokens <= 0) return HS_OK;
+  cudaError_t e = hs_launch(
+      hs::span_gather_kernel, dim3(n_requests * hs::LP_GATHER_BLOCKS + n_tokens), dim3(256), 0,
+      (cudaStream_t)stream, hs_pdl_enabled(), (__nv_bfloat16*)kv, (__nv_bfloat16*)q_out, base, q,
+      (const __nv_bfloat16*)pool, table, req_start, req_len, tok_pos, tok_req, n_requests, cap_rows,
+      window, max_single, H, G, D, V, (D + 63) / 64 * 64, page_size, num_pages, max_pages, status);
+  return e == cudaSuccess ? HS_OK : (int)e;
+}
+
+// kv [cap_rows, n_heads * (D + V)]: the expanded keys of all heads, then the values, and rope
+// [cap_rows, 64]; or (rope null) [cap_rows, kv_heads * (D + V)]: keys and values as span_gather left
+// them.  softcap 0 and sinks null: none.
 HS_EXPORT int hs_latent_prefill_tc(void* out, const void* q, const void* kv, const void* rope,
                                    const int* base, const int* plan, int tiles_off, int tile_cap,
                                    int n_tokens, int cap_rows, int n_heads, int D, int P, int V,
                                    int R, int window, float scale, const float* gate,
-                                   int gate_stride, int gate_off, int* status, void* stream) {
+                                   int gate_stride, int gate_off, int kv_heads, float softcap,
+                                   const float* sinks, int* status, void* stream) {
   using namespace hs;
   if (gate && (gate_off < 0 || gate_off + n_heads * V > gate_stride)) return HS_ERR_ARGUMENT;
-  if (!out || !q || !kv || !rope || !base || !plan || !status) return HS_ERR_ARGUMENT;
-  if (!hs_latent_prefill_tc_takes(D, P, V, R, window, scale) || n_heads <= 0)
+  if (!out || !q || !kv || !base || !plan || !status || softcap < 0.f) return HS_ERR_ARGUMENT;
+  if (n_heads <= 0 || kv_heads <= 0 || n_heads % kv_heads ||
+      (rope ? kv_heads != n_heads || !hs_latent_prefill_tc_takes(D, P, V, R, window, scale)
+            : !hs_span_prefill_tc_takes(n_heads, kv_heads, D, V, window, scale)))
     return HS_ERR_UNSUPPORTED;
   if (((uintptr_t)out | (uintptr_t)q | (uintptr_t)kv | (uintptr_t)rope) & 15) return HS_ERR_UNSUPPORTED;
   if (tile_cap <= 0 || n_tokens <= 0) return HS_OK;
-  const int nk = (D + 63) / 64 + 1, nv = (V + 63) / 64;
+  const int nk = (D + 63) / 64 + (rope ? 1 : 0), nv = (V + 63) / 64;
   CUtensorMap mq, mkv, mr;
   if (int e = lp_map(&mq, q, n_tokens, (long long)n_heads * nk * 64)) return e;
-  if (int e = lp_map(&mkv, kv, cap_rows, (long long)n_heads * (D + V))) return e;
-  if (int e = lp_map(&mr, rope, cap_rows, 64)) return e;
+  if (int e = lp_map(&mkv, kv, cap_rows, (long long)kv_heads * (D + V))) return e;
+  if (int e = rope ? lp_map(&mr, rope, cap_rows, 64) : HS_OK) return e;
+  if (!rope) mr = mkv;                                   // never used
   LatentTcParams p;
   p.out = (__nv_bfloat16*)out; p.plan = plan; p.base = base; p.status = status;
   p.tiles_off = tiles_off; p.n_heads = n_heads; p.D = D; p.V = V;
   p.window = window > 0 ? window : 1 << 28;
+  p.kv_group = n_heads / kv_heads; p.v_col = kv_heads * D; p.softcap = softcap; p.sinks = sinks;
   p.gate = gate; p.gate_stride = gate_stride; p.gate_off = gate_off;
   p.cap_rows = cap_rows; p.scale = scale;
   const dim3 grid(n_heads, tile_cap), block(LP_THREADS);
   cudaError_t e = cudaSuccess;
-#define HS_LP(NK, NV)                                                                             \
+#define HS_LP(NK, NV, T)                                                                          \
   do {                                                                                            \
-    auto kern = latent_prefill_tc_kernel<NK, NV>;                                                 \
+    auto kern = latent_prefill_tc_kernel<NK, NV, T>;                                              \
     /* more than half of an SM's shared memory: two of these never share an SM, since each       \
        allocates all of its tensor memory */                                                      \
     const size_t need = (size_t)(3 * NK + NV + 2) * LP_CHUNK + 256 + 1024;                        \
@@ -537,10 +668,19 @@ HS_EXPORT int hs_latent_prefill_tc(void* out, const void* q, const void* kv, con
     if (e == cudaSuccess)                                                                         \
       e = hs_launch(kern, grid, block, smem, (cudaStream_t)stream, false, mq, mkv, mr, p);        \
   } while (0)
-  if (nk == 2 && nv == 1) HS_LP(2, 1);
-  else if (nk == 2) HS_LP(2, 2);
-  else if (nv == 1) HS_LP(3, 1);
-  else HS_LP(3, 2);
+  if (rope) {
+    if (nk == 2 && nv == 1) HS_LP(2, 1, true);
+    else if (nk == 2) HS_LP(2, 2, true);
+    else if (nv == 1) HS_LP(3, 1, true);
+    else HS_LP(3, 2, true);
+  } else {
+    if (nk == 1 && nv == 1) HS_LP(1, 1, false);
+    else if (nk == 1) HS_LP(1, 2, false);
+    else if (nk == 2 && nv == 1) HS_LP(2, 1, false);
+    else if (nk == 2) HS_LP(2, 2, false);
+    else if (nv == 1) HS_LP(3, 1, false);
+    else HS_LP(3, 2, false);
+  }
 #undef HS_LP
   return e == cudaSuccess ? HS_OK : (int)e;
 }

@@ -207,7 +207,9 @@ def _declare(lib) -> None:
         "hs_latent_decode_mma": [P] * 7 + [I] * 7 + [F, I, I, I, P, P, I, I, P],
         "hs_latent_prefill_tc_takes": [I, I, I, I, I, F],
         "hs_latent_gather": [P] * 11 + [I] * 13 + [P, I, P, P],
-        "hs_latent_prefill_tc": [P] * 6 + [I] * 10 + [F, P, I, I, P, P],
+        "hs_latent_prefill_tc": [P] * 6 + [I] * 10 + [F, P, I, I, I, F, P, P, P],
+        "hs_span_prefill_tc_takes": [I, I, I, I, I, F],
+        "hs_span_gather": [P] * 10 + [I] * 12 + [P, P],
         "hs_latent_append": [P, P, P, P, P, P, I, I, I, I, I, F, I, I, I, I, P, P, I, P, P, I, I,
                              P],
         "hs_latent_attention": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, P, I,
@@ -363,6 +365,7 @@ class CudaOps:
         self.pooled_mma = True      # ... and of the attention over a window and pooled blocks
         self.ssm_chunk_rows = 64    # from this many tokens a step on
         self.ssm_chunks = True      # prompt portions of a state-space recurrence as chunks likewise
+        self.span_dense = True      # prompt portions of the latter on tcgen05, over gathered rows
         self.span_decode_mma = True     # single-query tokens of the latter likewise, where more than
         self.span_decode_keys = 512     # so many keys may be visible (measured: 128 blocks on the
         #                                 CUDA cores are through with 256 keys before the clusters)
@@ -1349,8 +1352,8 @@ class CudaOps:
         _check(self.lib.hs_latent_prefill_tc(
             _ptr(out), _ptr(q), _ptr(kv), _ptr(rope), _ptr(base), _ptr(plan.data),
             4 + plan_decode_ints(plan.n_rows), plan.tile_cap, T, rows, n_heads, dim, rot_dim, vdim,
-            rank, int(window), float(scale), _ptr(gate), g_stride, int(gate_offset), _ptr(status),
-            self._stream()), f"latent_prompt_attention(dim={dim},rot_dim={rot_dim},vdim={vdim})")
+            rank, int(window), float(scale), _ptr(gate), g_stride, int(gate_offset), n_heads, 0.0,
+            None, _ptr(status), self._stream()), f"latent_prompt_attention(dim={dim},rot_dim={rot_dim},vdim={vdim})")
 
     # -- the gated delta rule ---------------------------------------------------------------
     @staticmethod
@@ -2228,14 +2231,16 @@ class CudaOps:
 
     def span_attention(self, out, q, pool, table, tok_pos, tok_req, *, n_heads, n_kv_heads,
                        head_dim, value_dim, scale, slopes, window, keep_first, gate, gate_offset,
-                       out_scale, page_size, status, plan=None, softcap=0.0, sinks=None):
+                       out_scale, page_size, status, plan=None, softcap=0.0, sinks=None,
+                       req_start=None, req_len=None):
         """Per token at position i and query head h: softmax over the keys j <= i with
         i - j < window (0: all) or j < keep_first of (q . k) * scale - slopes[h] * (i - j)
         (``slopes`` float32 [heads] or None), with ``softcap`` c bent to c * tanh(score / c);
         with ``sinks`` (float32 [heads]) the denominator also holds exp(sinks[h]); the head's output times sigmoid(gate[t,
         gate_offset + h * value_dim + e]) (``gate`` float32 [T, *] or None) times
         ``out_scale``.  With the step's ``plan`` and a bfloat16 cache the plan's tiles (prompt
-        portions) run on the tensor cores, and so do its single-query tokens when many keys may be
+        portions) run on the tensor cores (with ``req_start`` and ``req_len``, no slopes, no kept
+        first rows and no scale, on tcgen05 over rows gathered from their pages), and so do its single-query tokens when many keys may be
         visible, with queries and weights in several bfloat16 terms (float32's mantissa), a cluster
         of blocks a token;
         without a plan, in float32 and for sizes the tile kernel does not take every token
@@ -2265,9 +2270,31 @@ class CudaOps:
         per_page = G * page_size * (D + V)
         num_pages = pool.numel() // per_page
         listed = head = None
-        if (plan is not None and plan.tile_cap > 0 and out.dtype == torch.bfloat16
+        d = plan.data if plan is not None else None
+        dense = self._span_dense_rows(plan, T, req_start, H, G, D, V, scale, slopes, window, keep_first,
+                                      out_scale) if out.dtype == torch.bfloat16 else 0
+        if dense:
+            pad, R = -(-D // 64) * 64, req_start.shape[0]
+            kv = self._scratch_buffer("span_rows", dense * G * (D + V), torch.bfloat16)
+            qp = self._scratch_buffer("span_queries", T * H * pad, torch.bfloat16)
+            base = self._scratch_buffer("span_base", R, torch.int32)
+            self.launches += 2
+            _check(self.lib.hs_span_gather(
+                _ptr(kv), _ptr(qp), _ptr(base), _ptr(q), _ptr(pool), _ptr(table), _ptr(req_start),
+                _ptr(req_len), _ptr(tok_pos), _ptr(tok_req), R, T, dense, int(window),
+                DECODE_MAX_NEW, H, G, D, V, int(page_size), num_pages, table.shape[1], _ptr(status),
+                self._stream()), f"span_gather(head_dim={D},value_dim={V})")
+            _check(self.lib.hs_latent_prefill_tc(
+                _ptr(out), _ptr(qp), _ptr(kv), None, _ptr(base), _ptr(d),
+                4 + plan_decode_ints(plan.n_rows), plan.tile_cap, T, dense, H, D, 0, V, 0,
+                int(window), float(scale), _ptr(gate), g_stride, int(gate_offset), G,
+                float(softcap), _ptr(sinks), _ptr(status), self._stream()),
+                f"span_attention(head_dim={D},value_dim={V})")
+            if plan.decode_cap == 0:
+                return
+            listed, head, T = d[4:], d, plan.decode_cap
+        elif (plan is not None and plan.tile_cap > 0 and out.dtype == torch.bfloat16
                 and self.tensor_cores and self.span_mma and plan.n_rows >= T):
-            d = plan.data
             code = self.lib.hs_span_attention_prefill(
                 _ptr(out), _ptr(q), _ptr(pool), _ptr(table), table.shape[1], num_pages,
                 _ptr(d[4 + plan_decode_ints(plan.n_rows):]), _ptr(d), plan.tile_cap,
@@ -2303,6 +2330,19 @@ class CudaOps:
             T, H, G, D, V, int(window), int(keep_first), float(scale), int(page_size),
             _DT[pool.dtype], _DT[out.dtype], _ptr(listed), _ptr(head), float(softcap), _ptr(sinks),
             _ptr(status), self._stream()), f"span_attention(head_dim={D},value_dim={V})")
+
+    def _span_dense_rows(self, plan, T, req_start, H, G, D, V, scale, slopes, window, keep_first,
+                         out_scale) -> int:
+        """Rows of the dense block with which the plan's prompt portions run on the tcgen05 kernel,
+        or 0 when they do not."""
+        if (plan is None or plan.tile_cap <= 0 or req_start is None or not self.tensor_cores
+                or not self.span_dense or slopes is not None or keep_first or out_scale != 1.0
+                or plan.n_rows < T
+                or not self.lib.hs_span_prefill_tc_takes(H, G, D, V, int(window), float(scale))):
+            return 0
+        rows = plan.n_rows + min(req_start.shape[0], plan.tile_cap) * (window - 1) if window \
+            else plan.prompt_rows
+        return rows if 2 * rows * G * (D + V) <= self.LATENT_EXPANDED_BYTES else 0
 
     # -- several copies of the stream --------------------------------------------------------
     def hyper_mix(self, dst, src, y=None, *, streams, mix=None, write=None, read=None, u=None,

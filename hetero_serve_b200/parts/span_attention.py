@@ -66,6 +66,8 @@ class SpanAttention(Mixer):
         self.rot_base, self.rot_dims, self.softcap = float(rot_base), int(rot_dims), float(softcap)
         self.values_are_keys, self.gate = bool(values_are_keys), bool(gate)
         self.out_scale, self.shares_cache, self.p = float(out_scale), bool(shares_cache), prefix
+        # without a window, prompts over gathered rows need one for every position they see
+        self.counts_prompt_rows = self.window == 0 and slopes is None
 
     def tensor_requests(self):
         p, W = self.p, self.width
@@ -141,7 +143,8 @@ class SpanAttention(Mixer):
                            scale=self.scale, slopes=self.slopes, window=self.window,
                            keep_first=self.keep_first, gate=proj if self.gate else None,
                            gate_offset=self.g_off or 0, out_scale=self.out_scale,
-                           softcap=self.softcap, sinks=self.sinks,
+                           softcap=self.softcap, sinks=self.sinks, req_start=ctx.req_start,
+                           req_len=ctx.req_len,
                            plan=getattr(ctx, "plan", None), **sizes)
         ops.linear(x, att, self.w_out, None, residual=None if fresh else x)
 

@@ -758,7 +758,8 @@ class PlainOps:
 
     def span_attention(self, out, q, pool, table, tok_pos, tok_req, *, n_heads, n_kv_heads,
                        head_dim, value_dim, scale, slopes, window, keep_first, gate, gate_offset,
-                       out_scale, page_size, status, plan=None, softcap=0.0, sinks=None):
+                       out_scale, page_size, status, plan=None, softcap=0.0, sinks=None,
+                       req_start=None, req_len=None):
         H, G, D, V = n_heads, n_kv_heads, head_dim, value_dim
         pv = pool.view(-1, G, page_size, D + V)
         for t in range(out.shape[0]):

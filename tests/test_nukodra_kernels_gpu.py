@@ -102,12 +102,12 @@ def _plain_attention(rows, H, G, D, V, offs, wq, wk, rot, scale, window, cap, si
     (6, 2, 48, 48, 70, 48, 0.0, True), (6, 2, 96, 96, 96, 96, 30.0, True),
     (20, 1, 64, 128, 33, 0, 10.0, True), (2, 1, 112, 80, 130, 112, 30.0, True),
     (16, 4, 72, 104, 64, 24, 12.0, True), (4, 2, 256, 64, 40, 128, 30.0, True)])
-@pytest.mark.parametrize("planned", ["no", "yes", "clusters"])
+@pytest.mark.parametrize("planned", ["no", "yes", "clusters", "dense"])
 def test_span_attention(ops, monkeypatch, dtype, tol, H, G, D, V, window, rot, cap, sinks, planned):
     """Two requests whose pages are scattered over the pool, in portions that end inside pages and
     windows; then single tokens.  Every position is compared.  The pages behind the window are
     taken out of the table: nothing may look them up.  Unused rows of the pool are NaN.  With the
-    step's work lists portions run as tiles; "clusters": single tokens on the kernel for many keys,
+    step's work lists portions run as tiles, "dense": over rows gathered from their pages; "clusters": single tokens on the kernel for many keys,
     whose products keep float32's mantissa, whatever the window."""
     if planned == "clusters":
         monkeypatch.setattr(ops, "span_decode_keys", 0)
@@ -158,9 +158,10 @@ def test_span_attention(ops, monkeypatch, dtype, tol, H, G, D, V, window, rot, c
         out = torch.full((T, H * V), float("nan"), dtype=dtype, device=DEV)
         work = ops.make_plan([(row, row, fed[r], k) for row, (r, k) in enumerate(step)], T, page) \
             if planned != "no" else None
+        more = dict(req_start=ints(starts), req_len=ints(k for _r, k in step)) if planned == "dense" else {}
         ops.span_attention(out, q, pool, tab, tok_pos, tok_req, scale=scale, slopes=None,
                            window=window, keep_first=0, gate=proj, gate_offset=g_off, out_scale=1.0,
-                           plan=work, softcap=cap, sinks=sk, **sizes)
+                           plan=work, softcap=cap, sinks=sk, **more, **sizes)
         at = 0
         for r, k in step:
             close(out[at:at + k], want[r][fed[r]:fed[r] + k], tol)
