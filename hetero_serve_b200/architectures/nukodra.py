@@ -1,6 +1,6 @@
 """Nukodra: a decoder whose layers are listed one by one in config.json.  The residual stream
 exists in several copies (hyper-connections): every sublayer reads a learned combination of them
-through an RMS norm whose weight is stored around zero, and writes its output and a learned mixture
+through an RMS norm whose weights are kept as offsets from one, and writes its output and a learned mixture
 of the copies back; the head reads their sum.  A layer is a mixer followed by a dense gated
 feed-forward (``W_down (silu(W_gate h) * (W_up h))``), or a mixer alone.  Three mixers:
 
@@ -218,7 +218,7 @@ def build_spec(cfg: NukodraConfig) -> ModelSpec:
 def init_weights(cfg: NukodraConfig, seed: int, shapes_only: bool = False):
     """Seeded random float32 weights under the checkpoint's names, drawn from one CPU generator
     in the order the names are listed here.  Matrices ~ N(0, 1/sqrt(in)); norm weights around 0
-    where they are stored so and around 1 elsewhere; connections near reading the mean of the
+    where they are offsets and around 1 elsewhere; connections near reading the mean of the
     copies, keeping each and writing to all, spread enough that an exchanged index shows."""
     gen = torch.Generator(device="cpu")
     gen.manual_seed(int(seed))

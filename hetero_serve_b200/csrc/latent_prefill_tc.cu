@@ -1,8 +1,8 @@
-// Attention over a shared latent for prompt portions, with or without a window, on tcgen05 tensor cores (sm_100a),
-// bfloat16 operands, float32 accumulators.  Same mathematics as latent_attention.cu, in the form
-// that costs prompts least: keys and values are EXPANDED per head, once for every position the
-// step's portions can see, instead of absorbing the expansions into the queries (a query and key
-// meet in dim + rot_dim and vdim numbers here, in 2 * kv_rank + rot_dim there).
+// Attention over a shared latent for prompt portions, with or without a window, on tcgen05 tensor
+// cores (sm_100a), bfloat16 operands, float32 accumulators.  Same mathematics as latent_attention.cu,
+// in the form that costs prompts least: keys and values are EXPANDED per head, once for every
+// position the step's portions can see, instead of absorbing the expansions into the queries (a query
+// and key meet in dim + rot_dim and vdim numbers here, in 2 * kv_rank + rot_dim there).
 //
 //   gather   the rows [latent | turned key part] of the positions a portion sees are brought from
 //            their pages into a dense block (latents and key parts apart), and the portion's

@@ -38,7 +38,7 @@ def unit_rms(x, eps):
 
 
 def layer_rms(x, weight, eps):
-    """The norm in front of a sublayer and of the head: its weight is stored around zero."""
+    """The norm in front of a sublayer and of the head: its weight is an offset from one."""
     return unit_rms(x, eps) * (1.0 + weight)
 
 

@@ -99,7 +99,7 @@ def _plain_attention(rows, H, G, D, V, offs, wq, wk, rot, scale, window, cap, si
     (4, 2, 26, 18, 21, 14, 15.0, True), (1, 1, 32, 32, 9, 32, 1.0, True),
     (2, 2, 8, 6, 1, 2, 0.0, True), (8, 2, 64, 64, 48, 64, 30.0, True),
     (4, 4, 128, 128, 40, 64, 20.0, False), (3, 1, 20, 258, 0, 20, 5.0, True),
-    (6, 2, 48, 48, 70, 48, 0.0, True), (6, 2, 96, 96, 96, 96, 30.0, True),
+    (6, 2, 48, 48, 70, 48, 0.0, True), (10, 2, 96, 96, 90, 64, 25.0, True),
     (20, 1, 64, 128, 33, 0, 10.0, True), (2, 1, 112, 80, 130, 112, 30.0, True),
     (16, 4, 72, 104, 64, 24, 12.0, True), (4, 2, 256, 64, 40, 128, 30.0, True)])
 @pytest.mark.parametrize("planned", ["no", "yes", "clusters", "dense"])
@@ -314,7 +314,7 @@ def _walk(xbc, dt, w, skip, H, G, N, V, state=None):
 
 
 SSM_SIZES = [(6, 2, 14, 10, 3), (4, 4, 8, 8, 1), (1, 1, 1, 8, 2), (5, 1, 9, 7, 5), (8, 2, 64, 32, 4),
-             (3, 1, 128, 64, 4), (4, 2, 48, 32, 3), (2, 1, 200, 96, 4), (4, 1, 16, 128, 4), (2, 2, 256, 16, 2),
+             (3, 1, 128, 64, 4), (4, 2, 80, 32, 3), (2, 1, 200, 96, 4), (4, 1, 16, 128, 4), (2, 2, 256, 16, 2),
              (2, 1, 500, 12, 4)]
 
 
